@@ -8,11 +8,6 @@
 //                   multiplied by a slice of the token's row in a table (a per-layer token input)
 #include "common.cuh"
 
-__device__ __forceinline__ float ts_gelu_tanh(float z) {
-  const float k = 0.7978845608028654f;  // sqrt(2/pi)
-  return 0.5f * z * (1.f + tanhf(k * (z + 0.044715f * z * z * z)));
-}
-
 template <typename TA>
 __global__ void gelu_tanh_kernel(const TA* __restrict__ x, TA* __restrict__ out, size_t n) {
   ts_pdl_prologue();

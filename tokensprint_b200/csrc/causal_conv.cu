@@ -4,6 +4,9 @@
 //   out[t, ch] = act(c + bias[ch])            mode CONV_PLAIN
 //   out[t, ch] = x[t, ch] + c                 mode CONV_ADD_INPUT (a sublayer that reads its input plus the convolution of it)
 //
+// `in_bias` (may be null) is added to every input row before anything else: the bias of the product
+// that made the rows, which the zeros before a sequence's start do not get.
+//
 // with act = silu or nothing.  The weights come tap by tap, [K, C] (what a checkpoint stores as [C, K] is
 // transposed once when it is loaded): the threads of a warp then read one tap's weights of neighbouring
 // channels from one line (channel by channel, every lane met a line of its own at every load, and the
@@ -23,7 +26,7 @@
 
 template <typename TI, typename TO>
 __global__ void causal_conv_kernel(const TI* __restrict__ xin, long long ld, const float* __restrict__ taps_w, const float* __restrict__ bias,
-                                   int K, float* __restrict__ conv_state, long long slot_stride, const int* __restrict__ state_slots,
+                                   const float* __restrict__ in_bias, int K, float* __restrict__ conv_state, long long slot_stride, const int* __restrict__ state_slots,
                                    const int* __restrict__ cu_seqlens, const int* __restrict__ seq_index, TO* __restrict__ out, long long ld_out,
                                    int T, int C, int act, int add_input) {
   ts_pdl_prologue();
@@ -39,13 +42,14 @@ __global__ void causal_conv_kernel(const TI* __restrict__ xin, long long ld, con
     const int first = t - t_begin, n = t_end - t_begin;
     if (first > 0 && first < K - 1) continue;  // worked out by the thread of the portion's first token
     float* st = conv_state + (size_t)state_slots[b] * slot_stride;  // [K-1, C]: the inputs before the portion, oldest first
+    const float xb = in_bias ? in_bias[col] : 0.f;
     const int count = first == 0 ? max(1, min(K - 1, n)) : 1;
     for (int tt = t; tt < t + count; ++tt) {
       float acc = bias ? bias[col] : 0.f;
       float cur = 0.f;
       for (int j = 0; j < K; ++j) {
         const int p = tt - (K - 1) + j;
-        const float in = p >= t_begin ? ts_to_float(xin[(size_t)p * ld + col]) : st[(size_t)(K - 1 + p - t_begin) * C + col];
+        const float in = p >= t_begin ? ts_to_float(xin[(size_t)p * ld + col]) + xb : st[(size_t)(K - 1 + p - t_begin) * C + col];
         acc = fmaf(taps_w[(size_t)j * C + col], in, acc);
         cur = in;
       }
@@ -56,7 +60,7 @@ __global__ void causal_conv_kernel(const TI* __restrict__ xin, long long ld, con
     if (first == 0)
       for (int j = 0; j < K - 1; ++j) {  // entry j becomes the input at position t_end - (K-1) + j
         const int p = t_end - (K - 1) + j;
-        st[(size_t)j * C + col] = p >= t_begin ? ts_to_float(xin[(size_t)p * ld + col]) : st[(size_t)(j + n) * C + col];
+        st[(size_t)j * C + col] = p >= t_begin ? ts_to_float(xin[(size_t)p * ld + col]) + xb : st[(size_t)(j + n) * C + col];
       }
   }
 }
@@ -90,15 +94,15 @@ __device__ __forceinline__ void conv_store8(__nv_bfloat16* p, const float (&v)[8
 
 template <typename TI, typename TO>
 __global__ void __launch_bounds__(128) causal_conv_vec_kernel(const TI* __restrict__ xin, long long ld, const float* __restrict__ taps_w,
-                                                              const float* __restrict__ bias, int K, float* __restrict__ conv_state,
-                                                              long long slot_stride, const int* __restrict__ state_slots,
+                                                              const float* __restrict__ bias, const float* __restrict__ in_bias, int K,
+                                                              float* __restrict__ conv_state, long long slot_stride, const int* __restrict__ state_slots,
                                                               const int* __restrict__ cu_seqlens, const int* __restrict__ seq_index,
                                                               TO* __restrict__ out, long long ld_out, int C, int act, int add_input) {
   ts_pdl_prologue();
   const int t = blockIdx.x, col = (blockIdx.y * 128 + threadIdx.x) * 8;
   if (col >= C) return;
   const int b = seq_index[t];
-  float acc[8], cur[8], w[8];
+  float acc[8], cur[8], w[8], xb[8];
   if (b < 0) {
 #pragma unroll
     for (int i = 0; i < 8; ++i) acc[i] = 0.f;
@@ -109,13 +113,20 @@ __global__ void __launch_bounds__(128) causal_conv_vec_kernel(const TI* __restri
   const int first = t - t_begin, n = t_end - t_begin;
   if (first > 0 && first < K - 1) return;  // worked out by the thread of the portion's first token
   float* st = conv_state + (size_t)state_slots[b] * slot_stride;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) xb[i] = in_bias ? in_bias[col + i] : 0.f;
+  auto load_row = [&](int p) {
+    conv_load8(xin + (size_t)p * ld + col, cur);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) cur[i] += xb[i];
+  };
   const int count = first == 0 ? max(1, min(K - 1, n)) : 1;
   for (int tt = t; tt < t + count; ++tt) {
 #pragma unroll
     for (int i = 0; i < 8; ++i) acc[i] = bias ? bias[col + i] : 0.f;
     for (int j = 0; j < K; ++j) {
       const int p = tt - (K - 1) + j;
-      if (p >= t_begin) conv_load8(xin + (size_t)p * ld + col, cur);
+      if (p >= t_begin) load_row(p);
       else conv_load8(st + (size_t)(K - 1 + p - t_begin) * C + col, cur);
       conv_load8(taps_w + (size_t)j * C + col, w);
 #pragma unroll
@@ -131,35 +142,35 @@ __global__ void __launch_bounds__(128) causal_conv_vec_kernel(const TI* __restri
   if (first == 0)
     for (int j = 0; j < K - 1; ++j) {  // entry j becomes the input at position t_end - (K-1) + j
       const int p = t_end - (K - 1) + j;
-      if (p >= t_begin) conv_load8(xin + (size_t)p * ld + col, cur);
+      if (p >= t_begin) load_row(p);
       else conv_load8(st + (size_t)(j + n) * C + col, cur);
       conv_store8(st + (size_t)j * C + col, cur);
     }
 }
 
 template <typename TI, typename TO>
-static int conv_launch(const void* xin, long long ld, const float* taps_w, const float* bias, int K, float* conv_state,
+static int conv_launch(const void* xin, long long ld, const float* taps_w, const float* bias, const float* in_bias, int K, float* conv_state,
                        long long slot_stride, const int* state_slots, const int* cu_seqlens, const int* seq_index, void* out, long long ld_out,
                        int T, int C, int act, int add_input, cudaStream_t s) {
   const bool aligned = C % 8 == 0 && ld % 8 == 0 && ld_out % 8 == 0 && slot_stride % 4 == 0 &&
                        (((uintptr_t)xin | (uintptr_t)out | (uintptr_t)conv_state | (uintptr_t)taps_w) & 15) == 0;
   if (aligned)
-    return ts_launch(causal_conv_vec_kernel<TI, TO>, dim3(T, (C / 8 + 127) / 128), dim3(128), 0, s, (const TI*)xin, ld, taps_w, bias, K, conv_state,
+    return ts_launch(causal_conv_vec_kernel<TI, TO>, dim3(T, (C / 8 + 127) / 128), dim3(128), 0, s, (const TI*)xin, ld, taps_w, bias, in_bias, K, conv_state,
                      slot_stride, state_slots, cu_seqlens, seq_index, (TO*)out, ld_out, C, act, add_input);
   const long long total = (long long)T * C;
   const unsigned blocks = (unsigned)min((total + 255) / 256, (long long)148 * 32);
-  return ts_launch(causal_conv_kernel<TI, TO>, dim3(blocks), dim3(256), 0, s, (const TI*)xin, ld, taps_w, bias, K, conv_state, slot_stride,
+  return ts_launch(causal_conv_kernel<TI, TO>, dim3(blocks), dim3(256), 0, s, (const TI*)xin, ld, taps_w, bias, in_bias, K, conv_state, slot_stride,
                    state_slots, cu_seqlens, seq_index, (TO*)out, ld_out, T, C, act, add_input);
 }
 
-TS_EXPORT int ts_causal_conv(const void* xin, int in_dtype, long long ld, const float* taps_w, const float* bias, int K, float* conv_state,
-                             long long slot_stride, const int* state_slots, const int* cu_seqlens, const int* seq_index, void* out,
+TS_EXPORT int ts_causal_conv(const void* xin, int in_dtype, long long ld, const float* taps_w, const float* bias, const float* in_bias, int K,
+                             float* conv_state, long long slot_stride, const int* state_slots, const int* cu_seqlens, const int* seq_index, void* out,
                              int out_dtype, long long ld_out, int T, int C, int act, int add_input, void* stream) {
   if (T <= 0) return 0;
   if (C <= 0 || K < 1 || (act != CONV_ACT_NONE && act != CONV_ACT_SILU) || (K > 1 && conv_state == nullptr)) return TS_ERR_BAD_ARGUMENT;
   cudaStream_t s = (cudaStream_t)stream;
 #define CONV_CASE(TI, TO) \
-  return conv_launch<TI, TO>(xin, ld, taps_w, bias, K, conv_state, slot_stride, state_slots, cu_seqlens, seq_index, out, ld_out, T, C, act, add_input, s)
+  return conv_launch<TI, TO>(xin, ld, taps_w, bias, in_bias, K, conv_state, slot_stride, state_slots, cu_seqlens, seq_index, out, ld_out, T, C, act, add_input, s)
   if (in_dtype == TS_DTYPE_F32 && out_dtype == TS_DTYPE_F32) CONV_CASE(float, float);
   if (in_dtype == TS_DTYPE_F32 && out_dtype == TS_DTYPE_BF16) CONV_CASE(float, __nv_bfloat16);
   if (in_dtype == TS_DTYPE_BF16 && out_dtype == TS_DTYPE_F32) CONV_CASE(__nv_bfloat16, float);

@@ -113,6 +113,26 @@ __device__ __forceinline__ float ts_warp_max(float v) {
   return v;
 }
 
+// gelu in its tanh form, z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))).
+__device__ __forceinline__ float ts_gelu_tanh(float z) {
+  const float k = 0.7978845608028654f;  // sqrt(2/pi)
+  return 0.5f * z * (1.f + tanhf(k * (z + 0.044715f * z * z * z)));
+}
+// The same as z * sigmoid(2 sqrt(2/pi) (z + 0.044715 z^3)) with the fast exponential and division, for
+// results that are rounded to bfloat16.
+__device__ __forceinline__ float ts_gelu_tanh_fast(float z) {
+  const float t = 1.5957691216057308f * (z + 0.044715f * z * z * z);
+  return __fdividef(z, 1.f + __expf(-t));
+}
+
+// What the gate of a gated feed-forward passes through.
+#define TS_GLU_SILU 0
+#define TS_GLU_GELU_TANH 1
+__device__ __forceinline__ float ts_glu_gate(float g, int act) { return act == TS_GLU_GELU_TANH ? ts_gelu_tanh(g) : g / (1.f + expf(-g)); }
+__device__ __forceinline__ float ts_glu_gate_fast(float g, int act) {
+  return act == TS_GLU_GELU_TANH ? ts_gelu_tanh_fast(g) : __fdividef(g, 1.f + __expf(-g));
+}
+
 // Sum over a block of up to 1024 threads; every thread gets the result.
 // `scratch` holds 33 floats of shared memory.
 __device__ __forceinline__ float ts_block_sum(float v, float* scratch) {

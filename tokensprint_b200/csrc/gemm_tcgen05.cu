@@ -116,6 +116,8 @@ struct GemmArgs {
   __nv_bfloat16* xprime;         //   [M, ldh] bf16(hidden * norm_w)
   float* ssq_out;                //   [tiles, M] sums of squares of the new hidden rows, per tile of 128 columns
   long long ldh;
+  float branch_scale;            //   multiplies the product as it joins the stream
+  int glu_act;                   // EPI_SWIGLU: what the gate passes through (TS_GLU_*)
   // EPI_QK_ROPE (head size 128 = one tile per head; rows of W: nq query heads, nkv key heads, nkv value heads):
   __nv_bfloat16* q_out;          //   [M, nq * 128]
   __nv_bfloat16* k_cache;        //   [slots, nkv, 128]
@@ -251,8 +253,8 @@ __device__ __forceinline__ Range cta_range(const GemmArgs& a, int cta) {
 // products, rows of W down the 128).  Called by the 128 epilogue threads together.
 //   EPI_PLAIN with a row scale: out = rstd[m] * sum.
 //   EPI_SWIGLU: the tile's first 64 rows of W are gate rows and the last 64 the up rows of the
-//     same 64 outputs: out[m][64 t + j] = silu(rstd g) * (rstd u).
-//   EPI_RESIDUAL_NORM: hidden[m][n] += sum; xprime = bf16(hidden * norm_w[n]); ssq_out[t][m] =
+//     same 64 outputs: out[m][64 t + j] = act(rstd g) * (rstd u), act = silu or the tanh form of gelu.
+//   EPI_RESIDUAL_NORM: hidden[m][n] += branch_scale * sum; xprime = bf16(hidden * norm_w[n]); ssq_out[t][m] =
 //     the sum over the tile's columns of hidden^2 (a warp takes a whole row of the tile, so
 //     the sum needs shuffles only and is the same in every run).
 // `ahead` (EPI_RESIDUAL_NORM): what this thread will need from device memory, asked for when the
@@ -307,7 +309,7 @@ __device__ __forceinline__ void fused_epilogue(const GemmArgs& args, int t, int 
       __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(args.out) + (size_t)m * args.ldo + t * 64 + j;
 #pragma unroll
       for (int i = 0; i < 4; ++i)
-        if (t * 64 + j + i < half_n) dst[i] = __float2bfloat16_rn(gs[i] / (1.f + __expf(-gs[i])) * us[i]);
+        if (t * 64 + j + i < half_n) dst[i] = __float2bfloat16_rn(ts_glu_gate_fast(gs[i], args.glu_act) * us[i]);
     }
   } else if (args.mode == EPI_RESIDUAL_NORM) {
     const int nl = (etid & 31) * 4, n0 = t * TILE_N + nl;  // the 32 lanes of a warp share m
@@ -324,7 +326,7 @@ __device__ __forceinline__ void fused_epilogue(const GemmArgs& args, int t, int 
       float ss = 0.f;
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        h[i] = old[i] + vals[i] * rstd[m];
+        h[i] = fmaf(args.branch_scale, vals[i] * rstd[m], old[i]);
         if (n0 + i < args.N) ss += h[i] * h[i];
       }
       float* hp = args.hidden + (size_t)m * args.ldh + n0;
@@ -1092,14 +1094,14 @@ TS_EXPORT int ts_wait_gives_up_probe(int* error, int limit, void* stream_) {
 //     that wrote it; every product row m is multiplied by rsqrt(sum_m / scale_width + scale_eps).
 //   mode 0: out as in ts_gemm_skinny_bf16.
 //   mode 1 (N even, rows of w in blocks of 128: 64 gate rows, then the 64 up rows of the same
-//     outputs): out [M, ldo] bf16 = silu(gate) * up, N / 2 columns.
-//   mode 2: hidden [M, ldh] float32 += product; xprime [M, ldh] bf16 = hidden * norm_w;
+//     outputs): out [M, ldo] bf16 = act(gate) * up, N / 2 columns; act by `glu_act`: silu or gelu (tanh form).
+//   mode 2: hidden [M, ldh] float32 += branch_scale * product; xprime [M, ldh] bf16 = hidden * norm_w;
 //     ssq_out [ceil(N / 128), M] = sums of squares of the new hidden rows per 128 columns.
 TS_EXPORT int ts_gemm_skinny_fused(const void* x, const void* w, void* out, int M, int N, int K, long long ldx,
                                    long long ldw, long long ldo, int out_f32, int mode, const float* scale_ssq,
                                    int scale_tiles, float scale_width, float scale_eps, float* hidden, long long ldh,
-                                   const float* norm_w, void* xprime, float* ssq_out, float* partial, int* counters,
-                                   int* error, const void* prefetch, long long prefetch_bytes, void* stream_);
+                                   const float* norm_w, void* xprime, float* ssq_out, float branch_scale, int glu_act, float* partial,
+                                   int* counters, int* error, const void* prefetch, long long prefetch_bytes, void* stream_);
 
 // The q/k/v projection of an attention layer with head size 128 (w: nq query heads, then nkv key
 // heads, then nkv value heads, 128 rows each), with what follows it done where each head's tile is
@@ -1120,7 +1122,7 @@ TS_EXPORT int ts_gemm_skinny_bf16(const void* x, const void* w, void* out, int M
                                   long long ldw, long long ldo, int out_f32, float* partial, int* counters,
                                   int* error, const void* prefetch, long long prefetch_bytes, void* stream_) {
   return ts_gemm_skinny_fused(x, w, out, M, N, K, ldx, ldw, ldo, out_f32, 0, nullptr, 0, 1.f, 0.f, nullptr, 0, nullptr,
-                              nullptr, nullptr, partial, counters, error, prefetch, prefetch_bytes, stream_);
+                              nullptr, nullptr, 1.f, TS_GLU_SILU, partial, counters, error, prefetch, prefetch_bytes, stream_);
 }
 
 // What every entry point shares: checks, the split of the work, tensor maps, launch.  `a` comes
@@ -1201,10 +1203,11 @@ TS_EXPORT int ts_gemm_chain_sync_words(void) { return (2 * MAX_PHASES + 1) * SYN
 TS_EXPORT int ts_gemm_skinny_fused(const void* x, const void* w, void* out, int M, int N, int K, long long ldx,
                                    long long ldw, long long ldo, int out_f32, int mode, const float* scale_ssq,
                                    int scale_tiles, float scale_width, float scale_eps, float* hidden, long long ldh,
-                                   const float* norm_w, void* xprime, float* ssq_out, float* partial, int* counters,
-                                   int* error, const void* prefetch, long long prefetch_bytes, void* stream_) {
+                                   const float* norm_w, void* xprime, float* ssq_out, float branch_scale, int glu_act, float* partial,
+                                   int* counters, int* error, const void* prefetch, long long prefetch_bytes, void* stream_) {
   if (M <= 0 || N <= 0) return 0;
   if (mode < 0 || mode > EPI_RESIDUAL_NORM) return TS_ERR_BAD_ARGUMENT;
+  if (glu_act != TS_GLU_SILU && glu_act != TS_GLU_GELU_TANH) return TS_ERR_BAD_ARGUMENT;
   if (mode == EPI_SWIGLU && ((N & 1) || out_f32 || ldo < N / 2)) return TS_ERR_BAD_ARGUMENT;
   if (mode == EPI_RESIDUAL_NORM && (hidden == nullptr || norm_w == nullptr || xprime == nullptr || ssq_out == nullptr || ldh < N))
     return TS_ERR_BAD_ARGUMENT;
@@ -1223,6 +1226,8 @@ TS_EXPORT int ts_gemm_skinny_fused(const void* x, const void* w, void* out, int 
   a.xprime = (__nv_bfloat16*)xprime;
   a.ssq_out = ssq_out;
   a.ldh = ldh;
+  a.branch_scale = branch_scale;
+  a.glu_act = glu_act;
   return run_gemm(x, w, M, N, K, ldx, ldw, a, partial, counters, error, prefetch, prefetch_bytes, stream_);
 }
 

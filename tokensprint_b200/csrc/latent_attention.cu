@@ -123,12 +123,14 @@ TS_EXPORT int ts_latent_prepare(const void* proj, int act_dtype, long long ld, i
 // against the absorbed query (all rank + rot entries), the warp agrees on the running max, then
 // all lanes walk the 32 rows together as values, each owning latent entries lane, lane + 32, ...
 // The order of a query's sums depends on its own keys only.  `gates` (one factor per token and
-// head, or null) multiplies the finished row.
+// head, or null) multiplies the finished row.  `sink` (one number per head, or null): exp(sink) joins
+// the denominator once, without a key or a value.
 template <typename TA>
 __global__ void latent_attention_simple_kernel(const TA* __restrict__ q_abs, const TA* __restrict__ cache, TA* __restrict__ out,
                                                const float* __restrict__ gates, const int* __restrict__ positions,
                                                const int* __restrict__ seq_index, const int* __restrict__ block_table,
-                                               int max_blocks, int page, int T, int H, int rank, int rot, float scale, int window) {
+                                               int max_blocks, int page, int T, int H, int rank, int rot, float scale, int window,
+                                               const float* __restrict__ sink) {
   ts_pdl_prologue();
   __shared__ float qs[LAS_WARPS][LAS_MAX_KEY_DIM];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -154,7 +156,8 @@ __global__ void latent_attention_simple_kernel(const TA* __restrict__ q_abs, con
   float acc[ACC];
 #pragma unroll
   for (int i = 0; i < ACC; ++i) acc[i] = 0.f;
-  float m = -INFINITY, l = 0.f;
+  // the sink is the first entry of the running maximum and sum
+  float m = sink ? sink[a] : -INFINITY, l = sink ? 1.f : 0.f;
   for (int base = lo; base <= p; base += 32) {
     const int j = base + lane;
     float s = -INFINITY;
@@ -195,7 +198,8 @@ __global__ void latent_attention_simple_kernel(const TA* __restrict__ q_abs, con
 
 TS_EXPORT int ts_latent_attention_simple(const void* q_abs, const void* cache, int act_dtype, void* out, const float* gates,
                                          const int* positions, const int* seq_index, const int* block_table, int max_blocks,
-                                         int page, int T, int H, int rank, int rot, float scale, int window, void* stream) {
+                                         int page, int T, int H, int rank, int rot, float scale, int window, const float* sink,
+                                         void* stream) {
   if (T <= 0) return 0;
   if (H <= 0 || rank <= 0 || rot < 0 || page <= 0 || max_blocks <= 0) return TS_ERR_BAD_ARGUMENT;
   if (rank + rot > LAS_MAX_KEY_DIM || rank > LAS_MAX_RANK) return TS_ERR_UNSUPPORTED_SIZE;
@@ -205,10 +209,10 @@ TS_EXPORT int ts_latent_attention_simple(const void* q_abs, const void* cache, i
   if (act_dtype == TS_DTYPE_F32)
     return ts_launch(latent_attention_simple_kernel<float>, dim3(blocks), dim3(LAS_WARPS * 32), 0, s, (const float*)q_abs,
                      (const float*)cache, (float*)out, gates, positions, seq_index, block_table, max_blocks, page, T, H, rank, rot,
-                     scale, window);
+                     scale, window, sink);
   if (act_dtype == TS_DTYPE_BF16)
     return ts_launch(latent_attention_simple_kernel<__nv_bfloat16>, dim3(blocks), dim3(LAS_WARPS * 32), 0, s,
                      (const __nv_bfloat16*)q_abs, (const __nv_bfloat16*)cache, (__nv_bfloat16*)out, gates, positions, seq_index,
-                     block_table, max_blocks, page, T, H, rank, rot, scale, window);
+                     block_table, max_blocks, page, T, H, rank, rot, scale, window, sink);
   return TS_ERR_BAD_ARGUMENT;
 }

@@ -1,6 +1,6 @@
 // Residual add + RMSNorm over the float32 residual stream.
 //
-//   h = hidden[row] (+ delta[row]);  hidden[row] = h (when a delta was added);
+//   h = hidden[row] (+ delta_scale * delta[row]);  hidden[row] = h (when a delta was added);
 //   out[r] = h * rsqrt(mean(h^2) + eps) * weight
 //
 // Sums, mean, rsqrt and the scaling are float32 with one rounding at the store, as in the
@@ -13,7 +13,7 @@
 template <typename TA>
 __global__ void add_rmsnorm_kernel(float* __restrict__ hidden, const TA* __restrict__ delta,
                                    const float* __restrict__ weight, TA* __restrict__ out,
-                                   const int* __restrict__ row_index, int H, float eps) {
+                                   const int* __restrict__ row_index, int H, float eps, float delta_scale) {
   ts_pdl_prologue();
   __shared__ float scratch[33];
   const int r = blockIdx.x;
@@ -26,7 +26,7 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ hidden, const TA* __restr
   float ss = 0.f;
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
     float v = h[i];
-    if (d) v += ts_to_float(d[i]);
+    if (d) v = fmaf(delta_scale, ts_to_float(d[i]), v);
     if (write_back) h[i] = v;
     ss += v * v;
   }
@@ -34,7 +34,7 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ hidden, const TA* __restr
   const float rstd = rsqrtf(ss / (float)H + eps);
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
     float v = h[i];
-    if (d && !write_back) v += ts_to_float(d[i]);
+    if (d && !write_back) v = fmaf(delta_scale, ts_to_float(d[i]), v);
     o[i] = ts_from_float<TA>(v * rstd * weight[i]);
   }
 }
@@ -63,7 +63,7 @@ __device__ __forceinline__ void ts_store4(__nv_bfloat16* p, float4 v) {
 template <typename TA>
 __global__ void add_rmsnorm_vec_kernel(float* __restrict__ hidden, const TA* __restrict__ delta,
                                        const float* __restrict__ weight, TA* __restrict__ out,
-                                       const int* __restrict__ row_index, int H, float eps) {
+                                       const int* __restrict__ row_index, int H, float eps, float delta_scale) {
   ts_pdl_prologue();
   __shared__ float scratch[33];
   const int r = blockIdx.x;
@@ -82,7 +82,10 @@ __global__ void add_rmsnorm_vec_kernel(float* __restrict__ hidden, const TA* __r
       v[k] = ts_load4(h + 4 * c);
       if (d) {
         const float4 dv = ts_load4(d + 4 * c);
-        v[k].x += dv.x; v[k].y += dv.y; v[k].z += dv.z; v[k].w += dv.w;
+        v[k].x = fmaf(delta_scale, dv.x, v[k].x);
+        v[k].y = fmaf(delta_scale, dv.y, v[k].y);
+        v[k].z = fmaf(delta_scale, dv.z, v[k].z);
+        v[k].w = fmaf(delta_scale, dv.w, v[k].w);
       }
     }
   }
@@ -108,52 +111,114 @@ __global__ void add_rmsnorm_vec_kernel(float* __restrict__ hidden, const TA* __r
 
 template <typename TA>
 static int launch_add_rmsnorm(float* hidden, const void* delta, const float* weight, void* out,
-                              const int* row_index, int rows, int H, float eps, cudaStream_t s) {
+                              const int* row_index, int rows, int H, float eps, float delta_scale, cudaStream_t s) {
   const int chunks = H >> 2;
   const bool aligned = (H % 4 == 0) && (((uintptr_t)hidden | (uintptr_t)delta | (uintptr_t)weight | (uintptr_t)out) % 16 == 0);
   if (aligned && chunks <= RN_MAX_CHUNKS * 1024) {
     int threads = (chunks + RN_MAX_CHUNKS - 1) / RN_MAX_CHUNKS;
     if (rows <= 512) threads = chunks;  // few rows: one piece per thread, shortest latency
     threads = min(1024, max(32, (threads + 31) / 32 * 32));
-    return ts_launch(add_rmsnorm_vec_kernel<TA>, dim3(rows), dim3(threads), 0, s, hidden, (const TA*)delta, weight, (TA*)out, row_index, H, eps);
+    return ts_launch(add_rmsnorm_vec_kernel<TA>, dim3(rows), dim3(threads), 0, s, hidden, (const TA*)delta, weight, (TA*)out, row_index, H, eps, delta_scale);
   } else {
     int threads = H >= 4096 ? 512 : (H >= 1024 ? 256 : (H >= 256 ? 128 : 64));
-    return ts_launch(add_rmsnorm_kernel<TA>, dim3(rows), dim3(threads), 0, s, hidden, (const TA*)delta, weight, (TA*)out, row_index, H, eps);
+    return ts_launch(add_rmsnorm_kernel<TA>, dim3(rows), dim3(threads), 0, s, hidden, (const TA*)delta, weight, (TA*)out, row_index, H, eps, delta_scale);
   }
 }
 
 TS_EXPORT int ts_add_rmsnorm(float* hidden, const void* delta, int act_dtype, const float* weight,
                              void* out, const int* row_index, int rows, int H, float eps,
-                             void* stream) {
+                             float delta_scale, void* stream) {
   if (rows <= 0) return 0;
   if (H <= 0) return TS_ERR_BAD_ARGUMENT;
   cudaStream_t s = (cudaStream_t)stream;
   if (act_dtype == TS_DTYPE_F32)
-    return launch_add_rmsnorm<float>(hidden, delta, weight, out, row_index, rows, H, eps, s);
+    return launch_add_rmsnorm<float>(hidden, delta, weight, out, row_index, rows, H, eps, delta_scale, s);
   if (act_dtype == TS_DTYPE_BF16)
-    return launch_add_rmsnorm<__nv_bfloat16>(hidden, delta, weight, out, row_index, rows, H, eps, s);
+    return launch_add_rmsnorm<__nv_bfloat16>(hidden, delta, weight, out, row_index, rows, H, eps, delta_scale, s);
   return TS_ERR_BAD_ARGUMENT;
 }
 
-// hidden[row] += delta[row] without a norm (the last residual sum when nothing follows it).
+// hidden[row] += scale * delta[row] without a norm (the last residual sum when nothing follows it).
 template <typename TA>
-__global__ void residual_add_kernel(float* __restrict__ hidden, const TA* __restrict__ delta, size_t n) {
+__global__ void residual_add_kernel(float* __restrict__ hidden, const TA* __restrict__ delta, size_t n, float scale) {
   ts_pdl_prologue();
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-  if (i < n) hidden[i] += ts_to_float(delta[i]);
+  if (i < n) hidden[i] = fmaf(scale, ts_to_float(delta[i]), hidden[i]);
 }
 
-TS_EXPORT int ts_residual_add(float* hidden, const void* delta, int act_dtype, long long n, void* stream) {
+TS_EXPORT int ts_residual_add(float* hidden, const void* delta, int act_dtype, long long n, float scale, void* stream) {
   if (n <= 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
   unsigned blocks = (unsigned)((n + 255) / 256);
   if (act_dtype == TS_DTYPE_F32)
-    return ts_launch(residual_add_kernel<float>, dim3(blocks), dim3(256), 0, s, hidden, (const float*)delta, (size_t)n);
+    return ts_launch(residual_add_kernel<float>, dim3(blocks), dim3(256), 0, s, hidden, (const float*)delta, (size_t)n, scale);
   else if (act_dtype == TS_DTYPE_BF16)
-    return ts_launch(residual_add_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, s, hidden, (const __nv_bfloat16*)delta, (size_t)n);
+    return ts_launch(residual_add_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, s, hidden, (const __nv_bfloat16*)delta, (size_t)n, scale);
   else
     return TS_ERR_BAD_ARGUMENT;
   return ts_launch_status();
+}
+
+// out[row] = in[row] * rsqrt(mean(in[row]^2) + eps) * weight on rows that are a column range of a wider
+// matrix (`ld` elements apart): the latent that queries pass, beside the other columns of its product.
+// A warp takes a row (short rows, many of them) and keeps nothing between its two passes: the second
+// one finds the row in the cache.
+template <typename TA>
+__global__ void __launch_bounds__(128) rmsnorm_rows_kernel(const TA* __restrict__ in, long long ld, const float* __restrict__ weight,
+                                                           TA* __restrict__ out, int rows, int width, float eps) {
+  ts_pdl_prologue();
+  const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= rows) return;
+  const TA* x = in + (size_t)row * ld;
+  float ss = 0.f;
+#pragma unroll 4
+  for (int i = lane; i < width; i += 32) {
+    const float v = ts_to_float(x[i]);
+    ss += v * v;
+  }
+  ss = ts_warp_sum(ss);
+  const float rstd = 1.f / sqrtf(ss / (float)width + eps);
+  TA* o = out + (size_t)row * width;
+#pragma unroll 4
+  for (int i = lane; i < width; i += 32) o[i] = ts_from_float<TA>(ts_to_float(x[i]) * rstd * weight[i]);
+}
+
+// The same, four entries per lane and access: widths and strides that are multiples of 4, bfloat16.
+__global__ void __launch_bounds__(128) rmsnorm_rows_vec_kernel(const __nv_bfloat16* __restrict__ in, long long ld,
+                                                               const float* __restrict__ weight, __nv_bfloat16* __restrict__ out,
+                                                               int rows, int width, float eps) {
+  ts_pdl_prologue();
+  const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= rows) return;
+  const __nv_bfloat16* x = in + (size_t)row * ld;
+  float ss = 0.f;
+#pragma unroll 4
+  for (int i = lane * 4; i < width; i += 128) {
+    const float4 v = ts_load4(x + i);
+    ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+  }
+  ss = ts_warp_sum(ss);
+  const float rstd = 1.f / sqrtf(ss / (float)width + eps);
+  __nv_bfloat16* o = out + (size_t)row * width;
+#pragma unroll 4
+  for (int i = lane * 4; i < width; i += 128) {
+    const float4 v = ts_load4(x + i), w = ts_load4(weight + i);
+    ts_store4(o + i, make_float4(v.x * rstd * w.x, v.y * rstd * w.y, v.z * rstd * w.z, v.w * rstd * w.w));
+  }
+}
+
+TS_EXPORT int ts_rmsnorm_rows(const void* in, int act_dtype, long long ld, const float* weight, void* out, int rows, int width, float eps,
+                              void* stream) {
+  if (rows <= 0) return 0;
+  if (width <= 0 || ld < width) return TS_ERR_BAD_ARGUMENT;
+  cudaStream_t s = (cudaStream_t)stream;
+  const dim3 grid((unsigned)((rows + 3) / 4)), block(128);
+  if (act_dtype == TS_DTYPE_F32)
+    return ts_launch(rmsnorm_rows_kernel<float>, grid, block, 0, s, (const float*)in, ld, weight, (float*)out, rows, width, eps);
+  if (act_dtype != TS_DTYPE_BF16) return TS_ERR_BAD_ARGUMENT;
+  if (width % 4 == 0 && ld % 4 == 0 && ((uintptr_t)in | (uintptr_t)out) % 8 == 0 && (uintptr_t)weight % 16 == 0)
+    return ts_launch(rmsnorm_rows_vec_kernel, grid, block, 0, s, (const __nv_bfloat16*)in, ld, weight, (__nv_bfloat16*)out, rows, width, eps);
+  return ts_launch(rmsnorm_rows_kernel<__nv_bfloat16>, grid, block, 0, s, (const __nv_bfloat16*)in, ld, weight, (__nv_bfloat16*)out, rows, width, eps);
 }
 
 // The norm on a branch's output, for layers that norm what a sublayer returns instead of what it

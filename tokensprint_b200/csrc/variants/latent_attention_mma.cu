@@ -19,7 +19,8 @@
 // (grid z), that leave unnormalised sums with their max and sum in scratch, and a second kernel
 // merges them.  Keys outside [position - window + 1, position] are masked per row; rows that are
 // not copied (outside the visible range, whose pages may be gone) are zeros in shared memory.
-// A query's sums depend on its own keys and on the split count only.
+// A query's sums depend on its own keys and on the split count only.  A learned score per head
+// (`sink`, or null) joins a row's sum once, where the row is finished.
 #include "../common.cuh"
 
 #ifndef TS_LAT_RANK
@@ -60,13 +61,16 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const unsigned (&a)[4], 
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
+// What a head's sink adds to a sum of exp2((score - m) * scale_log2).
+__device__ __forceinline__ float sink_term(float sink, float m, float scale_log2) { return exp2f(fmaf(sink, 1.4426950408889634f, -m * scale_log2)); }
 __device__ __forceinline__ void group_barrier(int group) { asm volatile("bar.sync %0, 128;" ::"r"(group + 1) : "memory"); }
 
 __global__ void __launch_bounds__(THREADS, 1) latent_attention_mma_kernel(
     const __nv_bfloat16* __restrict__ q_abs, const __nv_bfloat16* __restrict__ cache, __nv_bfloat16* __restrict__ out,
     const float* __restrict__ gates, const int* __restrict__ cu_seqlens, const int* __restrict__ context_lens,
     const int* __restrict__ block_table, int max_blocks, int page, int H, float scale_log2, int window, int splits,
-    float* __restrict__ part_o, float* __restrict__ part_m, float* __restrict__ part_l, long long total_rows) {
+    float* __restrict__ part_o, float* __restrict__ part_m, float* __restrict__ part_l, long long total_rows,
+    const float* __restrict__ sink) {
   ts_pdl_prologue();
   extern __shared__ __align__(16) unsigned char smem[];
   __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(smem);
@@ -281,7 +285,8 @@ __global__ void __launch_bounds__(THREADS, 1) latent_attention_mma_kernel(
       const int rr = r0 + row_local[r];
       if (rr >= rows_b) continue;
       const long long grow = grow0 + row_local[r];
-      const float f = l_run[r] > 0.f ? (gates ? gates[grow] : 1.f) / l_run[r] : 0.f;
+      const float l = sink ? l_run[r] + sink_term(sink[rr % H], m_run[r], scale_log2) : l_run[r];
+      const float f = l_run[r] > 0.f ? (gates ? gates[grow] : 1.f) / l : 0.f;
 #pragma unroll
       for (int i = 0; i < VT_W; ++i) {
         const int tile = vq * VT_W + i;
@@ -316,7 +321,8 @@ constexpr int MERGE_MAX_SPLITS = 64;
 
 __global__ void latent_attention_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_m,
                                               const float* __restrict__ part_l, __nv_bfloat16* __restrict__ out,
-                                              const float* __restrict__ gates, int splits, long long total_rows, float scale_log2) {
+                                              const float* __restrict__ gates, int splits, long long total_rows, float scale_log2,
+                                              const float* __restrict__ sink, int H) {
   ts_pdl_prologue();
   __shared__ float weight[MERGE_MAX_SPLITS];
   __shared__ float factor;
@@ -339,7 +345,7 @@ __global__ void latent_attention_merge_kernel(const float* __restrict__ part_o, 
     const float l = ts_warp_sum(w0 * l0 + w1 * l1);
     weight[lane] = w0;
     weight[lane + 32] = w1;
-    if (lane == 0) factor = l > 0.f ? g / l : 0.f;
+    if (lane == 0) factor = l > 0.f ? g / (sink ? l + sink_term(sink[row % H], m, scale_log2) : l) : 0.f;
   }
   __syncthreads();
   const float f = factor;
@@ -360,11 +366,13 @@ __global__ void latent_attention_merge_kernel(const float* __restrict__ part_o, 
 TS_EXPORT int ts_latent_attention_mma_rows() { return BM; }
 TS_EXPORT int ts_latent_attention_mma_keys() { return BN; }
 
-// q_abs [T, H, rank+rot] bf16; cache [slots, rank+rot] bf16; out [T, H, rank] bf16; gates [T, H] f32 or null.
+// q_abs [T, H, rank+rot] bf16; cache [slots, rank+rot] bf16; out [T, H, rank] bf16; gates [T, H] f32 or null;
+// sink [H] f32 or null.
 // scratch: splits * T * H * (rank + 2) floats when splits > 1.
 TS_EXPORT int ts_latent_attention_mma(const void* q_abs, const void* cache, void* out, const float* gates, const int* cu_seqlens,
                                       const int* context_lens, const int* block_table, int max_blocks, int page, int num_seqs,
-                                      int max_seqlen_q, int T, int H, float scale, int window, int splits, float* scratch, void* stream) {
+                                      int max_seqlen_q, int T, int H, float scale, int window, int splits, float* scratch,
+                                      const float* sink, void* stream) {
   if (num_seqs <= 0 || T <= 0) return 0;
   if (H <= 0 || page <= 0 || max_blocks <= 0 || max_seqlen_q <= 0 || splits < 1 || (splits > 1 && !scratch)) return TS_ERR_BAD_ARGUMENT;
   if (SMEM_BYTES > 227 * 1024 || num_seqs > 65535 || splits > MERGE_MAX_SPLITS) return TS_ERR_UNSUPPORTED_SIZE;
@@ -383,8 +391,8 @@ TS_EXPORT int ts_latent_attention_mma(const void* q_abs, const void* cache, void
   cudaStream_t s = (cudaStream_t)stream;
   int rc = ts_launch(latent_attention_mma_kernel, grid, dim3(THREADS), SMEM_BYTES, s, (const __nv_bfloat16*)q_abs, (const __nv_bfloat16*)cache,
                      (__nv_bfloat16*)out, gates, cu_seqlens, context_lens, block_table, max_blocks, page, H, scale_log2, window, splits,
-                     part_o, part_m, part_l, total_rows);
+                     part_o, part_m, part_l, total_rows, sink);
   if (rc != 0 || splits == 1) return rc;
   return ts_launch(latent_attention_merge_kernel, dim3((unsigned)total_rows), dim3(RANK >= 256 ? 256 : 64), 0, s, (const float*)part_o,
-                   (const float*)part_m, (const float*)part_l, (__nv_bfloat16*)out, gates, splits, total_rows, scale_log2);
+                   (const float*)part_m, (const float*)part_l, (__nv_bfloat16*)out, gates, splits, total_rows, scale_log2, sink, H);
 }

@@ -11,6 +11,7 @@ import tokensprint_b200.parts  # noqa: F401  (registers the built-in parts)
 from tokensprint_b200 import ops
 from tokensprint_b200.models.spec import ModelSpec
 from tokensprint_b200.parts.base import BuildContext, CacheNeed, LayerCache, Normed, PreNormed, Rounded, StepContext, TensorSpec, build_part
+from tokensprint_b200.parts.blocks import add_pending, norm_stream
 from tokensprint_b200.parts.linear import folding_possible, linear_float32_out, linear_scaled
 from tokensprint_b200.weights.loader import LoadedTensors, WeightSource, check_tensors
 
@@ -70,8 +71,10 @@ class Model:
                 raise ValueError(f"run {i} reads cache {keys[c]} that no run writes")
             need = self.blocks[run.layer].mixer.cache_need()
             w = plan[c].need
-            if (need.group_key, need.k_row, need.v_row, need.state_shape) != (w.group_key, w.k_row, w.v_row, w.state_shape):
-                raise ValueError(f"run {i} and run {plan[c].writer_run} share a cache but need different ones")
+            try:  # a reader may look further back than the run that fills the cache
+                plan[c] = CachePlanEntry(w.covering(need), plan[c].writer_run)
+            except ValueError as e:
+                raise ValueError(f"run {i} and run {plan[c].writer_run} share a cache but need different ones") from e
         self.cache_plan: list[CachePlanEntry] = [p for p in plan if p is not None]
         # An embedding transform that keeps something per request between steps gets a cache of its
         # own behind the runs' caches (writer_run -1: no run fills it); whoever binds device memory
@@ -167,8 +170,7 @@ class Model:
             if not last and order[i + 1].before is not None:
                 step.norm_after = None  # the stream changes once more before the next block's norm reads it
             if run.before is not None:
-                if isinstance(pending, torch.Tensor):  # the transform works on the complete stream
-                    ops.residual_add(hidden, pending)
+                add_pending(hidden, pending)  # the transform works on the complete stream
                 pending = None
                 transform = self.run_transforms[run.before]
                 if not transform.reads_through_ops:
@@ -213,7 +215,7 @@ class Model:
                 return linear_scaled(pending, self.head, float32_out=True)
             pending = None  # `hidden` is complete: norm it as usual
         normed = torch.empty((num_rows, self.spec.hidden_size), device=self.device, dtype=self.dtype)
-        self.final_norm.forward(hidden, pending, normed, row_index=rows)
+        norm_stream(self.final_norm, hidden, pending, normed, row_index=rows)
         return linear_float32_out(normed, self.head)
 
     def forward(self, step: StepContext, caches: list[LayerCache], rows: torch.Tensor, num_rows: int) -> torch.Tensor:

@@ -26,9 +26,10 @@ _c_ll = ctypes.c_longlong
 _SIGNATURES = {
     "ts_embed_gather": [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_void_p],
     "ts_feed_tokens": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p],
-    "ts_add_rmsnorm": [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_float, _c_void_p],
-    "ts_residual_add": [_c_void_p, _c_void_p, _c_int, _c_ll, _c_void_p],
-    "ts_swiglu": [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+    "ts_add_rmsnorm": [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_float, _c_float, _c_void_p],
+    "ts_residual_add": [_c_void_p, _c_void_p, _c_int, _c_ll, _c_float, _c_void_p],
+    "ts_rmsnorm_rows": [_c_void_p, _c_int, _c_ll, _c_void_p, _c_void_p, _c_int, _c_int, _c_float, _c_void_p],
+    "ts_swiglu": [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "ts_qk_norm_rope_store": [
         _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
         _c_float, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p,
@@ -48,7 +49,7 @@ _SIGNATURES = {
     "ts_latent_prepare": [_c_void_p, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_float,
                           _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void_p, _c_ll, _c_void_p],
     "ts_latent_attention_simple": [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
-                                   _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p],
+                                   _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_void_p],
     "ts_gelu_tanh": [_c_void_p, _c_void_p, _c_int, _c_ll, _c_void_p],
     "ts_capped_glu": [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_float, _c_void_p],
     "ts_gelu_gate_rows": [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_ll, _c_int, _c_int, _c_void_p],
@@ -266,8 +267,9 @@ def add_rmsnorm(
     out: torch.Tensor,
     eps: float,
     row_index: Optional[torch.Tensor] = None,
+    delta_scale: float = 1.0,
 ) -> None:
-    """hidden += delta (float32, in place) and out = RMSNorm(hidden) * weight.
+    """hidden += delta_scale * delta (float32, in place) and out = RMSNorm(hidden) * weight.
 
     hidden [T,H] f32; delta [T,H] of out's dtype or None; weight [H] f32; out [rows,H].
     With `row_index` ([rows] i32) only those rows are normed and hidden is left as it is.
@@ -292,22 +294,39 @@ def add_rmsnorm(
         raise KernelError("add_rmsnorm: out must have hidden's rows when no row_index is given")
     _check("add_rmsnorm", _fn("ts_add_rmsnorm")(
         hidden.data_ptr(), _ptr(delta), _act_code("out", out), weight.data_ptr(), out.data_ptr(),
-        _ptr(row_index), rows, H, float(eps), _stream()))
+        _ptr(row_index), rows, H, float(eps), float(delta_scale), _stream()))
 
 
-def residual_add(hidden: torch.Tensor, delta: torch.Tensor) -> None:
-    """hidden += delta in float32.  hidden [T,H] f32, delta [T,H] f32 or bf16."""
+def rmsnorm_rows(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: float) -> None:
+    """out = x * rsqrt(mean(x^2) + eps) * weight row by row, in float32; x [T, n] may be a column range of
+    a wider matrix, out [T, n] is of its type."""
+    flush_gemm_chain()
+    T, n = out.shape
+    _cuda_contig("out", out)
+    _cuda_contig("weight", weight, torch.float32)
+    _matrix_view("rmsnorm_rows: x", x, T, n, out.dtype)
+    if weight.numel() != n:
+        raise KernelError("rmsnorm_rows: weight must have one entry per column")
+    _check("rmsnorm_rows", _fn("ts_rmsnorm_rows")(x.data_ptr(), _act_code("x", x), x.stride(0), weight.data_ptr(), out.data_ptr(), T, n,
+                                                  float(eps), _stream()))
+
+
+def residual_add(hidden: torch.Tensor, delta: torch.Tensor, scale: float = 1.0) -> None:
+    """hidden += scale * delta in float32.  hidden [T,H] f32, delta [T,H] f32 or bf16."""
     flush_gemm_chain()
     _cuda_contig("hidden", hidden, torch.float32)
     _cuda_contig("delta", delta)
     if delta.shape != hidden.shape:
         raise KernelError("residual_add: shapes disagree")
     _check("residual_add", _fn("ts_residual_add")(
-        hidden.data_ptr(), delta.data_ptr(), _act_code("delta", delta), hidden.numel(), _stream()))
+        hidden.data_ptr(), delta.data_ptr(), _act_code("delta", delta), hidden.numel(), float(scale), _stream()))
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0) -> None:
-    """out[t,i] = silu(gate[t,i]) * up[t,i].  gate_up [T,2I], out [T,I].  block 0: gate i at column
+GLU_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
+
+
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0, activation: str = "silu") -> None:
+    """out[t,i] = act(gate[t,i]) * up[t,i], act = silu (SwiGLU) or the tanh form of gelu.  gate_up [T,2I], out [T,I].  block 0: gate i at column
     i, up at I + i; block 64: blocks of 128 columns, 64 gates and then their 64 ups."""
     flush_gemm_chain()
     _cuda_contig("gate_up", gate_up)
@@ -317,7 +336,8 @@ def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0) -> None:
         raise KernelError(f"swiglu: gate_up {tuple(gate_up.shape)} does not match out {tuple(out.shape)}")
     if block not in (0, 64) or (block and I % 64):
         raise KernelError(f"swiglu: block must be 0 or 64 (and then divide the width), got {block} for width {I}")
-    _check("swiglu", _fn("ts_swiglu")(gate_up.data_ptr(), out.data_ptr(), _act_code("out", out), T, I, int(block), _stream()))
+    _check("swiglu", _fn("ts_swiglu")(gate_up.data_ptr(), out.data_ptr(), _act_code("out", out), T, I, int(block), GLU_ACTIVATIONS[activation],
+                                      _stream()))
 
 
 QK_ROPE_MAX_HEAD_DIM = 512
@@ -521,6 +541,12 @@ def library_bmm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
     per-head products of a latent attention layer.  Strided views are taken as they are."""
     flush_gemm_chain()
     torch.bmm(a, w.transpose(1, 2), out=out)
+
+
+def library_bmm_float32(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+    """The same with a float32 result: the sums leave unrounded (gates that are worked out in 32-bit)."""
+    flush_gemm_chain()
+    torch.bmm(a, w.transpose(1, 2), out_dtype=torch.float32, out=out)
 
 
 def pair_hash_embed(hidden: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, positions: torch.Tensor, seq_index: torch.Tensor,
@@ -794,7 +820,7 @@ _SIGNATURES.update({
                        _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_float, _c_int,
                        _c_void_p],
     "ts_softcap_rows": [_c_void_p, _c_ll, _c_float, _c_void_p],
-    "ts_causal_conv": [_c_void_p, _c_int, _c_ll, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
+    "ts_causal_conv": [_c_void_p, _c_int, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                        _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "ts_delta_scan": [_c_void_p, _c_ll, _c_int, _c_int, _c_int, _c_void_p, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_ll, _c_void_p, _c_void_p,
                       _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_void_p],
@@ -1003,11 +1029,12 @@ CONV_ACTIVATIONS = {None: 0, "silu": 1}
 
 def causal_conv(xin: torch.Tensor, taps: torch.Tensor, bias: Optional[torch.Tensor], conv_state: Optional[torch.Tensor], state_slots: torch.Tensor,
                 cu_seqlens: torch.Tensor, seq_index: torch.Tensor, num_seqs: int, out: torch.Tensor, activation: Optional[str] = None,
-                add_input: bool = False) -> None:
+                add_input: bool = False, in_bias: Optional[torch.Tensor] = None) -> None:
     """A short causal convolution over time on every channel of xin [T, C] (a view of a wider matrix
     is fine): out[t] = act(sum_j taps[j] * x[t - (K-1) + j] + bias), or with `add_input`
     x[t] + that.  taps [K, C] float32, tap by tap (the last row weighs the current token; a checkpoint's
-    [C, K] is transposed once at load), bias [C] float32 or None.  conv_state [slots, >= (K-1)*C] float32 (a view with a row stride is fine) holds the last
+    [C, K] is transposed once at load), bias [C] float32 or None; in_bias [C] float32 or None is added to
+    every input row first (and not to the zeros before a sequence's start).  conv_state [slots, >= (K-1)*C] float32 (a view with a row stride is fine) holds the last
     K - 1 inputs of every request, oldest first; it is read for the inputs before a portion and then
     brought up to date with the portion's last inputs (K = 1: there is none, and conv_state may be None).
     Sums in float32; xin and out may differ in type."""
@@ -1021,6 +1048,10 @@ def causal_conv(xin: torch.Tensor, taps: torch.Tensor, bias: Optional[torch.Tens
         raise KernelError(f"causal_conv: taps must be [K, {C}], got {tuple(taps.shape)}")
     if bias is not None:
         _cuda_contig("bias", bias, torch.float32)
+    if in_bias is not None:
+        _cuda_contig("in_bias", in_bias, torch.float32)
+        if in_bias.numel() != C:
+            raise KernelError("causal_conv: in_bias must have one entry per channel")
     if K > 1 and (conv_state is None or conv_state.dtype != torch.float32 or conv_state.dim() != 2 or conv_state.stride(1) != 1
                   or conv_state.shape[1] < (K - 1) * C):
         raise KernelError(f"causal_conv: the state must be float32 [slots, >= {(K - 1) * C}]")
@@ -1028,9 +1059,54 @@ def causal_conv(xin: torch.Tensor, taps: torch.Tensor, bias: Optional[torch.Tens
     if activation not in CONV_ACTIVATIONS:
         raise KernelError(f"causal_conv: activation must be one of {list(CONV_ACTIVATIONS)}, got {activation!r}")
     _check("causal_conv", _fn("ts_causal_conv")(
-        xin.data_ptr(), _act_code("xin", xin), xin.stride(0), taps.data_ptr(), _ptr(bias), K, state_ptr, state_stride,
-        state_slots.data_ptr(), cu_seqlens.data_ptr(), seq_index.data_ptr(), out.data_ptr(), _act_code("out", out), out.stride(0), T, C,
+        xin.data_ptr(), _act_code("xin", xin), xin.stride(0), taps.data_ptr(), _ptr(bias), _ptr(in_bias), K, state_ptr,
+        state_stride, state_slots.data_ptr(), cu_seqlens.data_ptr(), seq_index.data_ptr(), out.data_ptr(), _act_code("out", out), out.stride(0), T, C,
         CONV_ACTIVATIONS[activation], 1 if add_input else 0, _stream()))
+
+
+_SIGNATURES["ts_rglru_scan"] = [
+    _c_void_p, _c_ll, _c_void_p, _c_ll, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_ll,
+    _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p,
+]
+
+
+def rglru_scan(u: torch.Tensor, pre: torch.Tensor, bias_r: torch.Tensor, bias_i: torch.Tensor, lam: torch.Tensor, decay_scale: float,
+               y: torch.Tensor, y_bias: Optional[torch.Tensor], state: torch.Tensor, state_slots: torch.Tensor, cu_seqlens: torch.Tensor,
+               seq_index: torch.Tensor, out: torch.Tensor, num_seqs: int, blocks: int, max_seqlen: int, decode_seqs: int = 0) -> None:
+    """The gated recurrence per channel over the tokens of every sequence, and the gelu of the second branch
+    (csrc/gated_recurrence.cu): with r, i = sigmoid(pre + bias), log a = -decay_scale r softplus(lam),
+    S <- a S + sqrt(1 - a^2) i u;  out = S gelu_tanh(y + y_bias).  u, y, out [T, w] of the compute type (row
+    strides are fine); pre [T, blocks, 2 w/blocks] float32: per block the r products, then the i products; biases and
+    lam [w] float32; state [slots, >= w] float32 (a view with a row stride is fine).  The first `decode_seqs`
+    sequences bring one token each."""
+    flush_gemm_chain()
+    T, w = out.shape
+    k = w // max(1, int(blocks))
+    _matrix_view("rglru_scan: u", u, T, w, out.dtype)
+    _matrix_view("rglru_scan: y", y, T, w, out.dtype)
+    _matrix_view("rglru_scan: out", out, T, w)
+    _cuda_contig("pre", pre, torch.float32)
+    for name, t in (("bias_r", bias_r), ("bias_i", bias_i), ("lam", lam)) + ((("y_bias", y_bias),) if y_bias is not None else ()):
+        _cuda_contig(name, t, torch.float32)
+        if t.numel() != w:
+            raise KernelError(f"rglru_scan: {name} must have one entry per channel")
+    if blocks < 1 or w % blocks or pre.numel() != T * 2 * w:
+        raise KernelError(f"rglru_scan: pre must be [{T}, {blocks}, {2 * k}] with blocks a divisor of {w}, got {tuple(pre.shape)}")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < w:
+        raise KernelError(f"rglru_scan: the state must be float32 [slots, >= {w}], got {tuple(state.shape)}")
+
+    def launch(tokens: int, first: int, count: int, single: int) -> None:
+        _check("rglru_scan", _fn("ts_rglru_scan")(
+            u.data_ptr(), u.stride(0), y.data_ptr(), y.stride(0), _act_code("out", out), pre.data_ptr(), bias_r.data_ptr(), bias_i.data_ptr(),
+            lam.data_ptr(), _ptr(y_bias), float(decay_scale), state.data_ptr(), state.stride(0), state_slots.data_ptr(), cu_seqlens.data_ptr(),
+            seq_index.data_ptr(), out.data_ptr(), out.stride(0), tokens, w, k, first, count, single, _stream()))
+
+    if max_seqlen <= 1:
+        launch(T, 0, num_seqs, 1)
+        return
+    if decode_seqs:
+        launch(decode_seqs, 0, decode_seqs, 1)
+    launch(T, decode_seqs, num_seqs - decode_seqs, 0)
 
 
 DELTA_MAX_KEY_DIM = 1024
@@ -1246,12 +1322,21 @@ def latent_prepare(proj: Optional[torch.Tensor], q_off: int, kv_off: int, gate_o
         0 if q_src is None else q_src.stride(0), _stream()))
 
 
+def _check_sink(name: str, sink: Optional[torch.Tensor], H: int) -> None:
+    if sink is not None:
+        _cuda_contig("sink", sink, torch.float32)
+        if sink.numel() != H:
+            raise KernelError(f"{name}: sink must have one entry per head")
+
+
 def latent_attention_simple(q_abs: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, gates: Optional[torch.Tensor],
                             positions: torch.Tensor, seq_index: torch.Tensor, block_table: torch.Tensor, page_size: int,
-                            num_heads: int, rank: int, rot_dim: int, scale: float, window: int = 0) -> None:
+                            num_heads: int, rank: int, rot_dim: int, scale: float, window: int = 0,
+                            sink: Optional[torch.Tensor] = None) -> None:
     """Causal attention of absorbed queries q_abs [T, H, rank+rot] over cached rows [pages, page,
     rank+rot] on CUDA cores: out [T, H, rank] = softmax(q_abs . row * scale) @ row[:rank], times
-    gates[t, h] if given.  Float32 or bfloat16; scores, softmax and sums in float32."""
+    gates[t, h] if given.  Float32 or bfloat16; scores, softmax and sums in float32.  `sink` [H] float32:
+    exp(sink[h]) joins every row's denominator."""
     flush_gemm_chain()
     _cuda_contig("q_abs", q_abs)
     _cuda_contig("cache", cache, q_abs.dtype)
@@ -1268,12 +1353,13 @@ def latent_attention_simple(q_abs: torch.Tensor, cache: torch.Tensor, out: torch
         raise KernelError(f"latent_attention_simple: the cache must be [pages, {page_size}, {D}], got {tuple(cache.shape)}")
     if gates is not None:
         _cuda_contig("gates", gates, torch.float32)
+    _check_sink("latent_attention_simple", sink, H)
     if block_table.dim() != 2 or positions.numel() < T or seq_index.numel() < T:
         raise KernelError("latent_attention_simple: block_table must be [B, max_blocks]; positions and seq_index need T entries")
     _check("latent_attention_simple", _fn("ts_latent_attention_simple")(
         q_abs.data_ptr(), cache.data_ptr(), _act_code("q_abs", q_abs), out.data_ptr(), _ptr(gates), positions.data_ptr(),
         seq_index.data_ptr(), block_table.data_ptr(), block_table.shape[1], page_size, T, H, int(rank), int(rot_dim), float(scale),
-        int(window), _stream()))
+        int(window), _ptr(sink), _stream()))
 
 
 def gelu_tanh(x: torch.Tensor, out: torch.Tensor) -> None:
@@ -1545,7 +1631,7 @@ def _latent_mma_fns(rank: int, rot_dim: int):
         lib = _build.load_variant("latent_attention_mma", {"TS_LAT_RANK": rank, "TS_LAT_ROT": rot_dim})
         fn = lib.ts_latent_attention_mma
         fn.argtypes = [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
-                       _c_int, _c_float, _c_int, _c_int, _c_void_p, _c_void_p]
+                       _c_int, _c_float, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p]
         fn.restype = _c_int
         for name in ("ts_latent_attention_mma_rows", "ts_latent_attention_mma_keys"):
             getattr(lib, name).restype = _c_int
@@ -1573,12 +1659,15 @@ def latent_attention_splits(device: torch.device, num_seqs: int, rows_per_seq: i
 
 def latent_attention_mma(q_abs: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, gates: Optional[torch.Tensor],
                          cu_seqlens: torch.Tensor, context_lens: torch.Tensor, block_table: torch.Tensor, page_size: int, num_seqs: int,
-                         max_seqlen_q: int, num_heads: int, rank: int, rot_dim: int, scale: float, window: int = 0, splits: int = 1) -> None:
+                         max_seqlen_q: int, num_heads: int, rank: int, rot_dim: int, scale: float, window: int = 0, splits: int = 1,
+                         sink: Optional[torch.Tensor] = None) -> None:
     """Causal attention of absorbed queries over cached rows on the tensor cores (bfloat16): q_abs
     [T, H, rank+rot] holds exactly the tokens of sequences 0..num_seqs-1 (cu_seqlens), cache [pages,
     page, rank+rot], out [T, H, rank] = softmax(q . row * scale) @ row[:rank] * gates.  `splits` > 1
-    cuts every sequence's keys into that many ranges (steps of few rows) merged by a second kernel."""
+    cuts every sequence's keys into that many ranges (steps of few rows) merged by a second kernel.  `sink`
+    [H] float32: exp(sink[h]) joins every row's denominator once."""
     flush_gemm_chain()
+    _check_sink("latent_attention_mma", sink, num_heads)
     _cuda_contig("q_abs", q_abs, torch.bfloat16)
     _cuda_contig("cache", cache, torch.bfloat16)
     _cuda_contig("out", out, torch.bfloat16)
@@ -1606,7 +1695,7 @@ def latent_attention_mma(q_abs: torch.Tensor, cache: torch.Tensor, out: torch.Te
     _check("latent_attention_mma", fn(
         q_abs.data_ptr(), cache.data_ptr(), out.data_ptr(), _ptr(gates), cu_seqlens.data_ptr(), context_lens.data_ptr(),
         block_table.data_ptr(), block_table.stride(0), page_size, num_seqs, max_seqlen_q, T, H, float(scale), int(window), int(splits),
-        _ptr(scratch), _stream()))
+        _ptr(scratch), _ptr(sink), _stream()))
     if splits > 1:
         global launch_count
         launch_count += 1  # the merge kernel
@@ -2240,7 +2329,7 @@ def gemm_skinny_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, prefet
 
 _SIGNATURES["ts_gemm_skinny_fused"] = [
     _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_ll, _c_ll, _c_ll, _c_int,
-    _c_int, _c_void_p, _c_int, _c_float, _c_float, _c_void_p, _c_ll, _c_void_p, _c_void_p, _c_void_p,
+    _c_int, _c_void_p, _c_int, _c_float, _c_float, _c_void_p, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_float, _c_int,
     _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_ll, _c_void_p,
 ]
 GEMM_FUSED_MAX_ROWS = 32
@@ -2261,6 +2350,8 @@ def gemm_skinny_fused(
     xprime: Optional[torch.Tensor] = None,
     ssq_out: Optional[torch.Tensor] = None,
     prefetch: Optional[torch.Tensor] = None,
+    branch_scale: float = 1.0,
+    activation: str = "silu",
 ) -> None:
     """x[M,K] @ w[N,K]^T on the tcgen05 tensor cores (M <= 32) with the work of the neighbouring
     small kernels done where each tile is finished.
@@ -2270,8 +2361,8 @@ def gemm_skinny_fused(
     the product is multiplied by rsqrt(sum_m / scale_width + scale_eps).
     mode GEMM_EPILOGUE_PLAIN: out[M,N] bf16 or float32.
     mode GEMM_EPILOGUE_SWIGLU: the rows of w come in blocks of 128, 64 gate rows and then the 64 up
-      rows of the same outputs; out[M,N/2] bf16 = silu(gate) * up.
-    mode GEMM_EPILOGUE_RESIDUAL_NORM: hidden[M,N] float32 += product; xprime[M,N] bf16 = hidden *
+      rows of the same outputs; out[M,N/2] bf16 = act(gate) * up (`activation`: one of GLU_ACTIVATIONS).
+    mode GEMM_EPILOGUE_RESIDUAL_NORM: hidden[M,N] float32 += branch_scale * product; xprime[M,N] bf16 = hidden *
       norm_weight; ssq_out[ceil(N/128), M] float32 = sums of squares of the new hidden rows.
     """
     if not gemm_skinny_supported(x, w) or x.shape[0] > GEMM_FUSED_MAX_ROWS:
@@ -2314,7 +2405,7 @@ def gemm_skinny_fused(
     _check_product("gemm_skinny_fused", _fn("ts_gemm_skinny_fused")(
         x.data_ptr(), w.data_ptr(), _ptr(out), M, N, K, x.stride(0), w.stride(0), ldo, out_f32,
         int(mode), _ptr(scale_ssq), scale_tiles, float(scale_width), float(scale_eps),
-        _ptr(hidden), N, _ptr(norm_weight), _ptr(xprime), _ptr(ssq_out),
+        _ptr(hidden), N, _ptr(norm_weight), _ptr(xprime), _ptr(ssq_out), float(branch_scale), GLU_ACTIVATIONS[activation],
         partial, counters, error,
         None if pf is None else pf.ptr, 0 if pf is None else min(pf.nbytes, GEMM_PREFETCH_BYTES),
         stream), x, w, out, scale_ssq, hidden, norm_weight, xprime, ssq_out)
@@ -2444,7 +2535,7 @@ _TIMED = ("embed_gather", "feed_tokens", "add_rmsnorm", "residual_add", "swiglu"
           "router_topk", "router", "moe_plan", "moe_gate_up", "moe_down", "moe_combine", "branch_norm_add", "stream_add",
           "qk_joint_norm_rope_store", "gla_scan", "gla_norm_gate", "linear_scan", "rows_dot_f32", "mlstm_gate_scan", "mlstm_norm_gate",
           "ssm_conv", "ssm_gate_norm", "scale_rows", "weighted_sum", "rope_table", "qkv_prepare", "gate_rows", "causal_conv", "delta_scan",
-          "softcap_rows")
+          "softcap_rows", "rglru_scan", "rmsnorm_rows", "library_bmm_float32")
 _plain_functions: dict[str, object] = {}
 _kernel_events: list[tuple[str, "torch.cuda.Event", "torch.cuda.Event"]] = []
 

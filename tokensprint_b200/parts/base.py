@@ -13,7 +13,7 @@ token belongs to, block tables, state slots) comes in a `StepContext`.
 
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Any, Callable, Mapping, Optional
 
 import torch
@@ -88,6 +88,20 @@ class CacheNeed:
     @property
     def group_key(self) -> tuple[str, int]:
         return (self.kind, self.window if self.kind in ("window", "chunk") else 0)
+
+    def covering(self, other: "CacheNeed") -> "CacheNeed":
+        """A need whose cache serves both: the same rows and state, and pages for as long as either may
+        still read them (the longer window; all keys where one of the two needs all)."""
+        if (self.k_row, self.v_row, self.state_shape) != (other.k_row, other.v_row, other.state_shape):
+            raise ValueError("the rows or the states differ")
+        if self.group_key == other.group_key:
+            return self
+        kinds = {self.kind, other.kind}
+        if not kinds <= {"full", "window"}:
+            raise ValueError(f"a cache cannot be both {self.kind!r} and {other.kind!r}")
+        if "full" in kinds:
+            return replace(self, kind="full", window=0)
+        return replace(self, window=max(self.window, other.window))
 
     @property
     def token_elements(self) -> int:
@@ -167,6 +181,7 @@ class ResidualNorm:
 
     hidden: torch.Tensor  # [T, width] float32, updated in place
     norm: NormParams
+    scale: float = 1.0  # multiplies the branch as it is added
 
 
 @dataclass
@@ -179,6 +194,15 @@ class PreNormed:
     ssq: torch.Tensor
     width: int
     eps: float
+
+
+@dataclass
+class Scaled:
+    """A branch output that is not yet added to the residual stream and is multiplied by a constant
+    when it is: what a block with a branch multiplier hands on in place of the plain tensor."""
+
+    x: torch.Tensor
+    factor: float
 
 
 @dataclass
@@ -243,6 +267,9 @@ class Part:
 
 
 class Norm(Part):
+    # True if forward() also takes `delta` as a Scaled (and multiplies it in float32 as it adds it).
+    adds_scaled = False
+
     def params(self) -> Optional[NormParams]:
         """The norm's weight, eps and width if it is a plain RMS norm that other parts may fold
         into their kernels; None keeps it a step of its own."""
@@ -255,7 +282,7 @@ class Norm(Part):
         out: torch.Tensor,
         row_index: Optional[torch.Tensor] = None,
     ) -> None:
-        """hidden (float32 residual) += delta if given; out = norm(hidden)."""
+        """hidden (float32 residual) += delta if given (a tensor, or a Scaled where `adds_scaled`); out = norm(hidden)."""
         raise NotImplementedError
 
     def forward_branch(self, branch: torch.Tensor, hidden: torch.Tensor, rounded: Optional[torch.Tensor] = None) -> None:

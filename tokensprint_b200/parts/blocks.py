@@ -17,6 +17,7 @@ from tokensprint_b200.parts.base import (
     PreNormed,
     ResidualNorm,
     Rounded,
+    Scaled,
     StepContext,
     TensorSpec,
     build_part,
@@ -24,20 +25,40 @@ from tokensprint_b200.parts.base import (
 )
 
 
+def add_pending(hidden: torch.Tensor, pending) -> None:
+    """Adds a branch output that is still waiting (a tensor or a Scaled) to the stream; nothing for anything else."""
+    if isinstance(pending, Scaled):
+        ops.residual_add(hidden, pending.x, pending.factor)
+    elif isinstance(pending, torch.Tensor):
+        ops.residual_add(hidden, pending)
+
+
+def norm_stream(norm, hidden: torch.Tensor, pending, out: torch.Tensor, row_index: Optional[torch.Tensor] = None) -> None:
+    """out = norm(hidden + pending): in one pass where the norm takes what is pending."""
+    if isinstance(pending, Scaled) and not norm.adds_scaled:
+        add_pending(hidden, pending)
+        pending = None
+    if row_index is None:
+        norm.forward(hidden, pending, out)
+    else:
+        norm.forward(hidden, pending, out, row_index=row_index)
+
+
 @register_part("block", "pre_norm")
 class PreNormBlock(Block):
-    """h = h + Mixer(Norm_a(h)); h = h + FeedForward(Norm_f(h))  (engine/nn/layers.py:111-121).
+    """h = h + s Mixer(Norm_a(h)); h = h + s FeedForward(Norm_f(h))  (engine/nn/layers.py:111-121, where s is 1).
 
     The residual stream is float32.  Each branch output is handed on as `pending` and
     added by the next norm in the same pass that norms it, so a residual sum never costs
     a pass over memory of its own.  A layer without a feed-forward ends with its mixer.
+    `residual_scale` (s) multiplies every branch output as it is added, in float32.
     """
 
     def __init__(self, ctx: BuildContext, *, mixer: PartSpec, mixer_norm: PartSpec, feed_forward: Optional[PartSpec] = None,
-                 ffn_norm: Optional[PartSpec] = None) -> None:
+                 ffn_norm: Optional[PartSpec] = None, residual_scale: float = 1.0) -> None:
         if (feed_forward is None) != (ffn_norm is None):
             raise ValueError("pre_norm block: a feed-forward and its norm come together")
-        self.dtype = ctx.dtype
+        self.dtype, self.residual_scale = ctx.dtype, float(residual_scale)
         self.mixer = build_part("mixer", mixer, ctx)
         self.feed_forward = None if feed_forward is None else build_part("feed_forward", feed_forward, ctx)
         self.mixer_norm = build_part("norm", mixer_norm, ctx)
@@ -80,26 +101,31 @@ class PreNormBlock(Block):
         else:
             x = torch.empty(hidden.shape, device=hidden.device, dtype=self.dtype)
             self._before(self.mixer_norm)
-            self.mixer_norm.forward(hidden, None if isinstance(pending, PreNormed) else pending, x)
+            norm_stream(self.mixer_norm, hidden, None if isinstance(pending, PreNormed) else pending, x)
+        next_norm = norm_after.params() if norm_after is not None else None
         if self.feed_forward is None:
             self._before(self.mixer)
-            return self.mixer.forward(x, step, cache)
+            if mixer_folds and next_norm is not None:
+                return self.mixer.forward(x, step, cache, fold=ResidualNorm(hidden, next_norm, self.residual_scale))
+            return self._pending(self.mixer.forward(x, step, cache))
         step.weight_after = self.feed_forward.first_weight()
         ffn_norm = self.ffn_norm.params()
         self._before(self.mixer)
         if mixer_folds and ffn_folds and ffn_norm is not None:
-            x = self.mixer.forward(x, step, cache, fold=ResidualNorm(hidden, ffn_norm))
+            x = self.mixer.forward(x, step, cache, fold=ResidualNorm(hidden, ffn_norm, self.residual_scale))
         else:
             mixed = self.mixer.forward(x, step, cache)
             x = torch.empty(hidden.shape, device=hidden.device, dtype=self.dtype)
             self._before(self.ffn_norm)
-            self.ffn_norm.forward(hidden, mixed, x)
+            norm_stream(self.ffn_norm, hidden, self._pending(mixed), x)
         step.weight_after = after_block
-        next_norm = norm_after.params() if norm_after is not None else None
         self._before(self.feed_forward)
         if ffn_folds and next_norm is not None:
-            return self.feed_forward.forward(x, step, fold=ResidualNorm(hidden, next_norm))
-        return self.feed_forward.forward(x, step)
+            return self.feed_forward.forward(x, step, fold=ResidualNorm(hidden, next_norm, self.residual_scale))
+        return self._pending(self.feed_forward.forward(x, step))
+
+    def _pending(self, branch: torch.Tensor):
+        return branch if self.residual_scale == 1.0 else Scaled(branch, self.residual_scale)
 
     @staticmethod
     def _before(part) -> None:
@@ -168,8 +194,8 @@ class PostNormBlock(Block):
         return x
 
     def forward(self, hidden, pending, step: StepContext, cache: LayerCache):
-        if isinstance(pending, torch.Tensor):  # a branch that the block before did not add
-            ops.residual_add(hidden, pending)
+        if isinstance(pending, (torch.Tensor, Scaled)):  # a branch that the block before did not add
+            add_pending(hidden, pending)
             pending = None
         x = self._rows(hidden, pending)
         after_block = step.weight_after
@@ -298,8 +324,8 @@ class SandwichNormBlock(Block):
 
     def forward(self, hidden, pending, step: StepContext, cache: LayerCache):
         after_block, norm_after = step.weight_after, step.norm_after
-        if isinstance(pending, torch.Tensor):  # a branch that the block before did not add
-            ops.residual_add(hidden, pending)
+        if isinstance(pending, (torch.Tensor, Scaled)):  # a branch that the block before did not add
+            add_pending(hidden, pending)
             pending = None
         if isinstance(pending, Normed):
             x = pending.x

@@ -1,4 +1,4 @@
-"""Dense SwiGLU feed-forward."""
+"""Dense gated feed-forward (SwiGLU, or with another activation of the gate)."""
 
 from __future__ import annotations
 
@@ -13,7 +13,8 @@ from tokensprint_b200.parts.linear import folding_possible, linear, linear_into_
 
 @register_part("feed_forward", "swiglu")
 class SwiGLUFeedForward(FeedForward):
-    """f = (silu(x Wg^T) * (x Wu^T)) Wd^T (engine/nn/layers.py:61-66), no biases.
+    """f = (act(x Wg^T) * (x Wu^T)) Wd^T (engine/nn/layers.py:61-66, with act = silu), no biases.
+    `activation`: "silu" (the default) or "gelu_tanh" (gelu in its tanh form).
 
     Gate and up weights are stacked at load into one [2I, H] matrix so one product
     gives both halves.  When the width allows it the rows are stacked in blocks of 64 gate rows
@@ -26,7 +27,11 @@ class SwiGLUFeedForward(FeedForward):
     reads_through_ops = True
     folds_norms = True
 
-    def __init__(self, ctx: BuildContext, *, hidden_size: int, intermediate_size: int, gate: str, up: str, down: str) -> None:
+    def __init__(self, ctx: BuildContext, *, hidden_size: int, intermediate_size: int, gate: str, up: str, down: str,
+                 activation: str = "silu") -> None:
+        if activation not in ops.GLU_ACTIVATIONS:
+            raise ValueError(f"swiglu feed-forward: activation must be one of {sorted(ops.GLU_ACTIVATIONS)}, got {activation!r}")
+        self.activation = activation
         self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
         self.names = {"gate": gate, "up": up, "down": down}
         self.gate_up: Optional[torch.Tensor] = None
@@ -64,11 +69,11 @@ class SwiGLUFeedForward(FeedForward):
         if not isinstance(x, torch.Tensor) and not own:
             raise ops.KernelError("swiglu feed-forward: a PreNormed input needs the engine's own GEMM for both products")
         if own:
-            act = linear_swiglu(x, self.gate_up, next_weight=self.down)
+            act = linear_swiglu(x, self.gate_up, next_weight=self.down, activation=self.activation)
         else:
             gu = linear(x, self.gate_up, next_weight=self.down)
             act = torch.empty((T, self.intermediate_size), device=gu.device, dtype=gu.dtype)
-            ops.swiglu(gu, act, self.block)
+            ops.swiglu(gu, act, self.block, self.activation)
         if fold is not None:
             if not own:
                 raise ops.KernelError("swiglu feed-forward: folding the residual sum needs the engine's own GEMM")

@@ -75,21 +75,22 @@ def linear_scaled(x: "PreNormed | torch.Tensor", weight: torch.Tensor, next_weig
     return out
 
 
-def linear_swiglu(x: "PreNormed | torch.Tensor", gate_up_blocks: torch.Tensor, next_weight: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """silu(x Wg^T) * (x Wu^T) in one kernel; the rows of `gate_up_blocks` come in blocks of 64
+def linear_swiglu(x: "PreNormed | torch.Tensor", gate_up_blocks: torch.Tensor, next_weight: Optional[torch.Tensor] = None,
+                  activation: str = "silu") -> torch.Tensor:
+    """act(x Wg^T) * (x Wu^T) in one kernel (act: silu or gelu_tanh); the rows of `gate_up_blocks` come in blocks of 64
     gate rows and the 64 up rows of the same outputs."""
     xt = x if isinstance(x, torch.Tensor) else x.x
     out = torch.empty((xt.shape[0], gate_up_blocks.shape[0] // 2), device=xt.device, dtype=xt.dtype)
     if isinstance(x, torch.Tensor):
-        ops.gemm_skinny_fused(x, gate_up_blocks, out=out, mode=ops.GEMM_EPILOGUE_SWIGLU, prefetch=next_weight)
+        ops.gemm_skinny_fused(x, gate_up_blocks, out=out, mode=ops.GEMM_EPILOGUE_SWIGLU, prefetch=next_weight, activation=activation)
     else:
         ops.gemm_skinny_fused(x.x, gate_up_blocks, out=out, mode=ops.GEMM_EPILOGUE_SWIGLU, scale_ssq=x.ssq, scale_width=x.width,
-                              scale_eps=x.eps, prefetch=next_weight)
+                              scale_eps=x.eps, prefetch=next_weight, activation=activation)
     return out
 
 
 def linear_into_residual(x: torch.Tensor, weight: torch.Tensor, fold: "ResidualNorm", next_weight: Optional[torch.Tensor] = None) -> "PreNormed":
-    """fold.hidden += x @ weight^T, and the input of the norm that follows, all in the product's
+    """fold.hidden += fold.scale * (x @ weight^T), and the input of the norm that follows, all in the product's
     kernel.  Returns the PreNormed that stands for norm(hidden)."""
     from tokensprint_b200.parts.base import PreNormed
 
@@ -97,7 +98,7 @@ def linear_into_residual(x: torch.Tensor, weight: torch.Tensor, fold: "ResidualN
     xprime = torch.empty((T, N), device=x.device, dtype=x.dtype)
     ssq = torch.empty((-(-N // 128), T), device=x.device, dtype=torch.float32)
     ops.gemm_skinny_fused(x, weight, mode=ops.GEMM_EPILOGUE_RESIDUAL_NORM, hidden=fold.hidden, norm_weight=fold.norm.weight,
-                          xprime=xprime, ssq_out=ssq, prefetch=next_weight)
+                          xprime=xprime, ssq_out=ssq, prefetch=next_weight, branch_scale=fold.scale)
     return PreNormed(xprime, ssq, fold.norm.width, fold.norm.eps)
 
 

@@ -7,7 +7,7 @@ from typing import Mapping, Optional
 import torch
 
 from tokensprint_b200 import ops
-from tokensprint_b200.parts.base import NormParams, BuildContext, Norm, TensorSpec, register_part
+from tokensprint_b200.parts.base import NormParams, BuildContext, Norm, Scaled, TensorSpec, register_part
 
 
 @register_part("norm", "rmsnorm")
@@ -21,6 +21,7 @@ class RMSNorm(Norm):
 
     graph_safe = True
     reads_through_ops = True
+    adds_scaled = True
 
     def __init__(self, ctx: BuildContext, *, dim: int, eps: float, weight: str, offset: float = 0.0, scalar: bool = False) -> None:
         self.dim, self.eps, self.weight_name, self.offset = int(dim), float(eps), weight, float(offset)
@@ -41,7 +42,10 @@ class RMSNorm(Norm):
         return NormParams(self.weight, self.eps, self.dim)
 
     def forward(self, hidden, delta, out, row_index=None) -> None:
-        ops.add_rmsnorm(hidden, delta, self.weight, out, self.eps, row_index)
+        scale = 1.0
+        if isinstance(delta, Scaled):
+            delta, scale = delta.x, delta.factor
+        ops.add_rmsnorm(hidden, delta, self.weight, out, self.eps, row_index, delta_scale=scale)
 
     def forward_branch(self, branch, hidden, rounded=None) -> None:
         ops.rmsnorm_add(branch, self.weight, hidden, self.eps, rounded)
