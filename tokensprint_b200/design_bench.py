@@ -24,6 +24,13 @@ two norms and behind a short convolution of its input) beside Dazilix, the close
 has (the same block arrangement, attention and a linear recurrence, routed experts), at equal width,
 depth, heads and expert sizes, with the distance of Vasosun's attention, recurrence and small kernels
 from their rooflines next to the like kernels of Dazilix.
+
+`python bench.py --designs mugulorn` runs Mugulorn (latent attention inside a window with sinks and an
+output gate, a layer that reads its cached rows, two gated recurrences per channel without a
+feed-forward, gelu feed-forwards) beside Vasosun, the closest design the engine has (the same latent
+attention, a recurrence), put together from the same kinds of layers at equal sizes: latent attention,
+its reader, two delta layers, dense feed-forwards where Mugulorn has them; with the distance of both
+designs' kernels from their rooflines.
 """
 
 from __future__ import annotations
@@ -155,6 +162,100 @@ def vasosun_config(s: dict) -> dict:
 def dazilix_beside_vasosun(s: dict) -> dict:
     d = next(v for k, v in DAZILIX_SIZES.items() if v["width"] == s["width"])
     return dazilix_config(d)
+
+
+# Mugulorn at the same widths: a latent attention of Vasosun's sizes (its window holds the prompt, so that it does the
+# work of Vasosun's), a second one that reads the first one's rows, and two recurrent layers without a feed-forward whose
+# channels are as many as the model's (blocks of 256, four taps); dense feed-forwards of the width of a real model's.
+# Vasosun beside it: the same two latent layers and two delta layers (heads of 64 x 128) without a feed-forward.
+MUGULORN_SIZES = {
+    "w2048": dict(width=2048, heads=16, layers=4, ff=6144, window=4096, kv_rank=512, rot_dim=64, q_rank=1536, lru=2048, blocks=8, taps=4,
+                  delta_dim=64, delta_vdim=128),
+    "w4096": dict(width=4096, heads=32, layers=4, ff=12288, window=4096, kv_rank=512, rot_dim=64, q_rank=3072, lru=4096, blocks=16, taps=4,
+                  delta_dim=64, delta_vdim=128),
+}
+
+
+def _latent_layer(s: dict) -> dict:
+    return {"heads": s["heads"], "dim": 128, "rot_dim": s["rot_dim"], "vdim": 128, "kv_rank": s["kv_rank"], "q_rank": s["q_rank"],
+            "scale": 192 ** -0.5, "rot": {"base": 1000000.0, "dims": s["rot_dim"],
+                                          "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+
+
+def mugulorn_config(s: dict) -> dict:
+    lat = dict(_latent_layer(s), mask={"size": s["window"]})
+    rec = {"type": "rglru", "mixer": {"width": s["lru"], "blocks": s["blocks"], "conv": s["taps"]}, "mlp": None}
+    mlp = {"kind": "dense", "ff": s["ff"]}
+    return {"architecture": "Mugulorn", "vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "residual_mult": 0.5, "layers": [{"type": "latent_attention", "mixer": lat, "mlp": mlp},
+                                             {"type": "latent_attention", "mixer": dict(lat, kv_from=0), "mlp": mlp}, rec, rec]}
+
+
+def vasosun_beside_mugulorn(s: dict) -> dict:
+    lat = _latent_layer(s)
+    delta = {"type": "delta", "mixer": {"heads": s["heads"], "kv_heads": s["heads"], "dim": s["delta_dim"], "vdim": s["delta_vdim"], "conv": s["taps"]},
+             "mlp": None}
+    mlp = {"kind": "dense", "ff": s["ff"]}
+    return {"architecture": "Vasosun", "vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-6}, "canon": {"taps": s["taps"]},
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 1000003, "mul_cur": 31}}, "logit_softcap": 30.0,
+            "layers": [{"type": "latent_attention", "mixer": lat, "mlp": mlp},
+                       {"type": "latent_attention", "mixer": dict(lat, kv_from=0), "mlp": mlp}, delta, delta]}
+
+
+def _mugulorn_rooflines(design: str, s: dict, m: dict, peaks: dict) -> dict[str, Any]:
+    """Both designs' kernels against their rooflines, from the per-class timers.  The latent attention: per
+    (query, key, head) 576 + 512 multiply-adds against the bf16 peak; a decode step reads every cached row once
+    per layer.  The recurrences: the gated one moves its inputs and its output once (per channel and token u, y,
+    the result in bf16 and, where they are not worked out in the kernel, two float32 gate products) against the
+    copy bandwidth; the delta rule costs 8 float32 operations per state entry and token against the FFMA rate in a
+    prompt, and moves every request's state in a decode step.  The small kernels move their inputs and outputs
+    once.  All entries are sums over the layers of a step."""
+    out: dict[str, Any] = {}
+    H, W, T = s["heads"], s["width"], PREFILL_TOKENS
+    hbm, bf16 = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    ffma_peak = 148 * 128 * 2 * peaks.get("sm_max_mhz", 1965.0) * 1e6
+    R, D, Q, w, ff = s["kv_rank"], s["kv_rank"] + s["rot_dim"], s["q_rank"], s["lru"], s["ff"]
+    delta_entries, chans = H * s["delta_dim"] * s["delta_vdim"], H * (2 * s["delta_dim"] + s["delta_vdim"])
+    gates_in_scan = "library_bmm_float32" not in m["prefill_kernels"]
+    if design == "mugulorn":
+        small = {  # bytes per token
+            "add_rmsnorm": 6 * W * 12, "causal_conv": 2 * w * (2 + 2), "rmsnorm_rows": 2 * Q * 4, "gate_rows": 2 * 3 * H * 128 * 2,
+            "latent_prepare": 2 * H * (192 + s["rot_dim"]) * 2 + 2 * D * 2, "swiglu": 2 * 3 * ff * 2,
+            "rglru_scan": 2 * w * (6 + (0 if gates_in_scan else 8)),
+        }
+    else:
+        small = {
+            "branch_norm_add": 6 * W * 12, "causal_conv": 6 * W * (2 + 2) + 2 * chans * (2 + 4), "rmsnorm_rows": 2 * Q * 4,
+            "gla_norm_gate": 2 * H * s["delta_vdim"] * 8, "latent_prepare": 2 * H * (192 + s["rot_dim"]) * 2 + 2 * D * 2, "swiglu": 2 * 3 * ff * 2,
+        }
+    steps = [("prefill", m["prefill_kernels"], T)] + [(f"decode_b{b}", m[f"decode_b{b}_kernels"], b) for b in DECODE_BATCHES]
+    for phase, kernels, tokens in steps:
+        for name, per_token in small.items():
+            ms = kernels.get(name, {}).get("ms", 0.0)
+            if ms > 0:
+                out[f"{phase}_{name}_ms"] = round(ms, 4)
+                if phase == "prefill":
+                    out[f"{phase}_{name}_of_hbm_peak"] = round(tokens * per_token / (ms * 1e-3) / hbm, 3)
+        ms = kernels.get("delta_scan", {}).get("ms", 0.0)
+        if ms > 0:
+            out[f"{phase}_delta_scan_ms"] = round(ms, 4)
+            if phase == "prefill":
+                out["prefill_delta_scan_of_ffma_peak"] = round(2 * 8.0 * T * delta_entries / (ms * 1e-3) / ffma_peak, 3)
+            else:
+                out[f"{phase}_delta_scan_of_hbm_peak"] = round(2 * tokens * delta_entries * 8 / (ms * 1e-3) / hbm, 3)
+        ms = kernels.get("rglru_step", {}).get("ms", 0.0)
+        if ms > 0:  # a decode step's recurrence with its gate products: their weights, the states, u, y and the result
+            moved = 2 * (2 * w * (w // s["blocks"]) * 2 + tokens * w * (8 + 6))
+            out[f"{phase}_rglru_step_ms"] = round(ms, 4)
+            out[f"{phase}_rglru_step_of_hbm_peak"] = round(moved / (ms * 1e-3) / hbm, 3)
+        ms = kernels.get("latent_attention_mma", {}).get("ms", 0.0)
+        if ms > 0:
+            out[f"{phase}_latent_attention_ms"] = round(ms, 4)
+            if phase == "prefill":
+                out["prefill_latent_attention_of_bf16_peak"] = round(2 * 2 * H * T * (T + 1) / 2 * (D + R) / (ms * 1e-3) / bf16, 3)
+            else:
+                out[f"{phase}_latent_attention_of_hbm_peak"] = round(2 * tokens * DECODE_CONTEXT * D * 2 / (ms * 1e-3) / hbm, 3)
+    return out
 
 
 def _vasosun_rooflines(s: dict, m: dict, peaks: dict) -> dict[str, Any]:
@@ -421,10 +522,12 @@ def run(steps: int, warmup: int, peaks: dict, which: str = "fegetar") -> dict[st
 
     result: dict[str, Any] = {"metric": "design_comparison", "dtype": "bf16", "data": "synthetic, random weights",
                               "prefill_tokens": PREFILL_TOKENS, "decode_context": DECODE_CONTEXT, "sizes": {}}
-    sizes = {"dazilix": DAZILIX_SIZES, "pekunex": PEKUNEX_SIZES, "vasosun": VASOSUN_SIZES}.get(which, SIZES)
+    sizes = {"dazilix": DAZILIX_SIZES, "pekunex": PEKUNEX_SIZES, "vasosun": VASOSUN_SIZES, "mugulorn": MUGULORN_SIZES}.get(which, SIZES)
     for name, s in sizes.items():
         row: dict[str, Any] = {"size": s}
-        if which == "vasosun":
+        if which == "mugulorn":
+            pair = (("mugulorn", mugulorn_config(s)), ("vasosun", vasosun_beside_mugulorn(s)))
+        elif which == "vasosun":
             pair = (("vasosun", vasosun_config(s)), ("dazilix", dazilix_beside_vasosun(s)))
         elif which == "pekunex":
             pair = (("pekunex", pekunex_config(s)), ("dazilix", dazilix_beside_pekunex(s)))
@@ -438,8 +541,11 @@ def run(steps: int, warmup: int, peaks: dict, which: str = "fegetar") -> dict[st
             m = _measure(model, steps, warmup)
             m["weight_bytes"] = model.weight_bytes()
             sd = DAZILIX_SIZES[name] if (which in ("pekunex", "vasosun") and design == "dazilix") else s
-            m.update(_attention_rooflines(design, sd, m, peaks))
-            if which == "vasosun":
+            if which != "mugulorn":
+                m.update(_attention_rooflines(design, sd, m, peaks))
+            if which == "mugulorn":
+                m.update(_mugulorn_rooflines(design, s, m, peaks))
+            elif which == "vasosun":
                 m.update(_vasosun_rooflines(s, m, peaks) if design == "vasosun" else _dazilix_rooflines(sd, m, peaks))
             elif which == "pekunex":
                 m.update(_pekunex_rooflines(s, m, peaks) if design == "pekunex" else _dazilix_rooflines(sd, m, peaks))

@@ -1109,6 +1109,45 @@ def rglru_scan(u: torch.Tensor, pre: torch.Tensor, bias_r: torch.Tensor, bias_i:
     launch(T, decode_seqs, num_seqs - decode_seqs, 0)
 
 
+_SIGNATURES["ts_rglru_step"] = [
+    _c_void_p, _c_ll, _c_void_p, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_ll, _c_void_p,
+    _c_void_p, _c_void_p, _c_ll, _c_int, _c_int, _c_int, _c_void_p,
+]
+
+
+def rglru_step_supported(u: torch.Tensor, gates: torch.Tensor) -> bool:
+    """Whether rglru_step takes these: bfloat16, block widths and rows on 16-byte boundaries."""
+    return (u.dtype == torch.bfloat16 and gates.dtype == torch.bfloat16 and gates.shape[2] % 8 == 0 and u.stride(0) % 8 == 0
+            and u.data_ptr() % 16 == 0 and gates.data_ptr() % 16 == 0)
+
+
+def rglru_step(u: torch.Tensor, gates: torch.Tensor, bias_r: torch.Tensor, bias_i: torch.Tensor, lam: torch.Tensor, decay_scale: float,
+               y: torch.Tensor, y_bias: Optional[torch.Tensor], state: torch.Tensor, state_slots: torch.Tensor, seq_index: torch.Tensor,
+               out: torch.Tensor) -> None:
+    """rglru_scan for a step in which every sequence brings one token, with the gate products (float32 sums)
+    in the same kernel: gates [blocks, 2 k, k] bfloat16, per block the r matrix and then the i matrix, both
+    [out, in]; the rest as rglru_scan takes it."""
+    flush_gemm_chain()
+    T, w = out.shape
+    _matrix_view("rglru_step: u", u, T, w, torch.bfloat16)
+    _matrix_view("rglru_step: y", y, T, w, torch.bfloat16)
+    _matrix_view("rglru_step: out", out, T, w, torch.bfloat16)
+    _cuda_contig("gates", gates, torch.bfloat16)
+    blocks, k = gates.shape[0], gates.shape[2]
+    if blocks * k != w or gates.shape[1] != 2 * k or not rglru_step_supported(u, gates):
+        raise KernelError(f"rglru_step: gates must be [blocks, 2 k, k] with blocks * k = {w} and k a multiple of 8, got {tuple(gates.shape)}")
+    for name, t in (("bias_r", bias_r), ("bias_i", bias_i), ("lam", lam)) + ((("y_bias", y_bias),) if y_bias is not None else ()):
+        _cuda_contig(name, t, torch.float32)
+        if t.numel() != w:
+            raise KernelError(f"rglru_step: {name} must have one entry per channel")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < w or seq_index.numel() < T:
+        raise KernelError(f"rglru_step: the state must be float32 [slots, >= {w}], got {tuple(state.shape)}, seq_index one entry per token")
+    _check("rglru_step", _fn("ts_rglru_step")(
+        u.data_ptr(), u.stride(0), y.data_ptr(), y.stride(0), gates.data_ptr(), bias_r.data_ptr(), bias_i.data_ptr(), lam.data_ptr(), _ptr(y_bias),
+        float(decay_scale), state.data_ptr(), state.stride(0), state_slots.data_ptr(), seq_index.data_ptr(), out.data_ptr(), out.stride(0), T, w, k,
+        _stream()))
+
+
 DELTA_MAX_KEY_DIM = 1024
 # TS_DELTA_LANES (for measurements): lanes that share a value column of the delta rule's state (a power of two up to 32);
 # unset or 0: the kernel's own choice by the key width
@@ -2535,7 +2574,7 @@ _TIMED = ("embed_gather", "feed_tokens", "add_rmsnorm", "residual_add", "swiglu"
           "router_topk", "router", "moe_plan", "moe_gate_up", "moe_down", "moe_combine", "branch_norm_add", "stream_add",
           "qk_joint_norm_rope_store", "gla_scan", "gla_norm_gate", "linear_scan", "rows_dot_f32", "mlstm_gate_scan", "mlstm_norm_gate",
           "ssm_conv", "ssm_gate_norm", "scale_rows", "weighted_sum", "rope_table", "qkv_prepare", "gate_rows", "causal_conv", "delta_scan",
-          "softcap_rows", "rglru_scan", "rmsnorm_rows", "library_bmm_float32")
+          "softcap_rows", "rglru_scan", "rglru_step", "rmsnorm_rows", "library_bmm_float32")
 _plain_functions: dict[str, object] = {}
 _kernel_events: list[tuple[str, "torch.cuda.Event", "torch.cuda.Event"]] = []
 

@@ -25,7 +25,7 @@ class GatedRecurrence(Mixer):
 
     One product gives [y | x]; the convolution adds x's bias as it reads its inputs (the zeros before a
     sequence get none); the block products leave float32 sums; one kernel does gates, recurrence and the
-    second branch's gelu.  Gates, decays, the state and the recurrence are float32 whatever the compute
+    second branch's gelu, and the block products too in a bfloat16 step of one token per sequence.  Gates, decays, the state and the recurrence are float32 whatever the compute
     dtype.  The state slot holds [width] states followed by the last taps - 1 inputs of the convolution
     [taps - 1, width], oldest first; zeros before the first token, so prompts may be cut anywhere.
 
@@ -87,12 +87,16 @@ class GatedRecurrence(Mixer):
         u = torch.empty((T, w), device=dev, dtype=dtype)
         ops.causal_conv(proj[:, w:], self.conv_weight, self.conv_bias, state[:, w:] if self.taps > 1 else None, step.state_slots,
                         step.cu_seqlens_q, step.seq_index, step.num_seqs, u, in_bias=self.x_bias)
-        pre = torch.empty((T, B, 2 * k), device=dev, dtype=torch.float32)
-        batched = ops.sgemm_nt_batched if dtype == torch.float32 else ops.library_bmm_float32
-        batched(u.view(T, B, k).transpose(0, 1), self.gate_weight, pre.transpose(0, 1))
         out = torch.empty((T, w), device=dev, dtype=dtype)
-        ops.rglru_scan(u, pre, self.r_bias, self.i_bias, self.lam, self.decay_scale, proj[:, :w], self.y_bias, state, step.state_slots,
-                       step.cu_seqlens_q, step.seq_index, out, step.num_seqs, B, step.max_seqlen_q, step.decode_seqs)
+        if step.max_seqlen_q == 1 and ops.rglru_step_supported(u, self.gate_weight):
+            ops.rglru_step(u, self.gate_weight, self.r_bias, self.i_bias, self.lam, self.decay_scale, proj[:, :w], self.y_bias, state,
+                           step.state_slots, step.seq_index, out)
+        else:
+            pre = torch.empty((T, B, 2 * k), device=dev, dtype=torch.float32)
+            batched = ops.sgemm_nt_batched if dtype == torch.float32 else ops.library_bmm_float32
+            batched(u.view(T, B, k).transpose(0, 1), self.gate_weight, pre.transpose(0, 1))
+            ops.rglru_scan(u, pre, self.r_bias, self.i_bias, self.lam, self.decay_scale, proj[:, :w], self.y_bias, state, step.state_slots,
+                           step.cu_seqlens_q, step.seq_index, out, step.num_seqs, B, step.max_seqlen_q, step.decode_seqs)
         if fold is not None:
             return linear_into_residual(out, self.o_weight, fold, next_weight=step.weight_after)
         return linear(out, self.o_weight, next_weight=step.weight_after)
