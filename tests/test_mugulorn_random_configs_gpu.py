@@ -28,8 +28,8 @@ def random_config(rng: random.Random) -> dict:
         return m
 
     def latent():
-        own = {"heads": rng.choice([1, 2, 3, 4, 8]), "dim": rng.choice([2, 8, 16, 24, 32, 40]), "vdim": rng.choice([4, 8, 12, 32, 64]),
-               "q_rank": rng.choice([6, 16, 24, 48, 96]), "scale": rng.choice([0.05, 0.1, 0.2])}
+        own = {"heads": rng.choice([1, 2, 3, 4, 8]), "dim": rng.choice([2, 8, 16, 24, 32, 40]), "vdim": rng.choice([4, 5, 8, 12, 32, 64]),
+               "q_rank": rng.choice([6, 7, 16, 24, 48, 96]), "scale": rng.choice([0.05, 0.1, 0.2])}
         if latents and rng.random() < 0.5:  # a reader: the source's latent width, rotated part and rotation; the rest its own
             j, src = rng.choice(latents)
             return {"type": "latent_attention", "mixer": mask(dict(src, **own, kv_from=j))}

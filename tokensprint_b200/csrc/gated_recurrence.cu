@@ -294,7 +294,36 @@ __global__ void __launch_bounds__(128) rglru_gate_step_kernel(RgParams P, const 
     for (int g = 0; g < 2; ++g)
 #pragma unroll
       for (int h = 0; h < 2; ++h) ahead[n][g][h] = weight(warp + 4 * n, g, h);
+  // what the step of this thread's four (token, channel) pairs will need beside the products: threads of a half
+  // warp take the 16 channels of one token.  The parameters come before the wait, the rest is asked for right
+  // behind it, so that these trips run beside those of the products' inputs.
+  const int ch = threadIdx.x & 15, c = block * k + row0 + ch;
+  const bool mine = row0 + ch < k;
+  float neg_rate = 0.f, br = 0.f, bi = 0.f, yb = 0.f;
+  if (mine) {
+    neg_rate = -P.decay_scale * rg_softplus(P.lam[c]);
+    br = P.bias_r[c];
+    bi = P.bias_i[c];
+    yb = P.y_bias ? P.y_bias[c] : 0.f;
+  }
   ts_pdl_wait();
+  float* slot[RG_STEP_TOKENS / 8];
+  float old[RG_STEP_TOKENS / 8], uv[RG_STEP_TOKENS / 8], yv[RG_STEP_TOKENS / 8];
+#pragma unroll
+  for (int i = 0; i < RG_STEP_TOKENS / 8; ++i) {
+    const int t = t0 + (threadIdx.x >> 4) + i * 8;
+    const int b = mine && t < P.T ? P.seq_index[t] : -1;
+    slot[i] = b >= 0 ? P.state + (size_t)P.state_slots[b] * P.slot_stride + c : nullptr;
+  }
+#pragma unroll
+  for (int i = 0; i < RG_STEP_TOKENS / 8; ++i) {
+    const int t = t0 + (threadIdx.x >> 4) + i * 8;
+    if (slot[i] != nullptr) {
+      old[i] = *slot[i];
+      uv[i] = __bfloat162float(u[(size_t)t * P.ld_u + c]);
+      yv[i] = __bfloat162float(y[(size_t)t * P.ld_y + c]);
+    }
+  }
 
   float acc[2][4][4];
 #pragma unroll
@@ -305,7 +334,6 @@ __global__ void __launch_bounds__(128) rglru_gate_step_kernel(RgParams P, const 
 #pragma unroll
     for (int n = 0; n < 4; ++n) {
       const int t = t0 + n * 8 + quad;
-      if (t0 + n * 8 >= P.T) break;  // the same for the whole warp
       const uint4 x = t < P.T && chunk * 32 + qi * 8 < k ? *reinterpret_cast<const uint4*>(u + (size_t)t * P.ld_u + (size_t)block * k + chunk * 32 + qi * 8) : zero;
 #pragma unroll
       for (int g = 0; g < 2; ++g) {
@@ -328,27 +356,20 @@ __global__ void __launch_bounds__(128) rglru_gate_step_kernel(RgParams P, const 
 #pragma unroll
       for (int e = 0; e < 4; ++e) part[warp][g][quad + (e >> 1) * 8][n * 8 + 2 * qi + (e & 1)] = acc[g][n][e];
   __syncthreads();
-  // threads of a half warp take the 16 channels of one token
-  const int ch = threadIdx.x & 15, c = block * k + row0 + ch;
-  if (row0 + ch >= k) return;
-  const float neg_rate = -P.decay_scale * rg_softplus(P.lam[c]), br = P.bias_r[c], bi = P.bias_i[c], yb = P.y_bias ? P.y_bias[c] : 0.f;
+  if (!mine) return;
 #pragma unroll
   for (int i = 0; i < RG_STEP_TOKENS / 8; ++i) {
     const int tt = (threadIdx.x >> 4) + i * 8, t = t0 + tt;
     if (t >= P.T) break;
-    const int b = P.seq_index[t];
     float o = 0.f;
-    if (b >= 0) {
-      float* s = P.state + (size_t)P.state_slots[b] * P.slot_stride + c;
-      const float old = *s;
-      const float uv = __bfloat162float(u[(size_t)t * P.ld_u + c]), yv = __bfloat162float(y[(size_t)t * P.ld_y + c]);
+    if (slot[i] != nullptr) {
       const float pr = part[0][0][ch][tt] + part[1][0][ch][tt] + (part[2][0][ch][tt] + part[3][0][ch][tt]);
       const float pi = part[0][1][ch][tt] + part[1][1][ch][tt] + (part[2][1][ch][tt] + part[3][1][ch][tt]);
       float a, x;
-      rg_gates_fast(pr + br, pi + bi, uv, neg_rate, a, x);
-      const float S = fmaf(a, old, x);
-      *s = S;
-      o = S * ts_gelu_tanh_fast(yv + yb);
+      rg_gates_fast(pr + br, pi + bi, uv[i], neg_rate, a, x);
+      const float S = fmaf(a, old[i], x);
+      *slot[i] = S;
+      o = S * ts_gelu_tanh_fast(yv[i] + yb);
     }
     out[(size_t)t * P.ld_out + c] = __float2bfloat16_rn(o);
   }
