@@ -17,8 +17,8 @@
 // The pairs are combined by shuffles inside a warp, then across the warps through shared memory (a warp per
 // channel, lanes over the warps), and each group then runs its tokens from the state that enters it.  So
 // every input is read once, gates are worked out once, and the dependent chain per round is a handful of
-// multiply-adds instead of one per token.  The next round's inputs are fetched before the current
-// round is worked on.  No CTA waits for another.
+// multiply-adds instead of one per token.  The next round's inputs are asked for as soon as
+// this round's gates are worked out.  No CTA waits for another.
 #include "common.cuh"
 
 #define RG_CH 16
