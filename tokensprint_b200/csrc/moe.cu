@@ -6,7 +6,9 @@
 //                 sigmoid(logit), handed on as they are or divided by their sum (`renormalize`), or
 //                 the softmax over the chosen logits alone (`score_mode`); or, with the softmax over all
 //                 logits as scores, the `top` largest of score + correction (a number per expert that
-//                 steers the choice only) with the scores themselves as weights.
+//                 steers the choice only) with the scores themselves as weights.  Experts may form equal groups of
+//                 neighbours: only those of the groups with the best members are then chosen.  A constant
+//                 may multiply the weights.
 //   moe_plan    : the (token, choice) pairs sorted by expert: offsets[e] .. offsets[e+1] are expert
 //                 e's places in `order` (pair indices), tile_offsets[e] its first row tile of
 //                 `tile_rows` places (64 for the kernels here, more for the tensor-core ones).
@@ -33,9 +35,17 @@
 #define MOE_MAX_EXPERTS 4096
 
 
-// The choice of one token by one warp: logits z [E] (shared or global memory), the bias already in.
+// What a router may do beyond scores and a choice of the largest.
+struct RouterGroups {
+  int count;    // experts form `count` equal groups of neighbours (0 or 1: no groups)
+  int keep;     // only experts of the `keep` groups whose best member is largest may be chosen
+  float scale;  // a constant on every weight, after they are divided by their sum
+};
+
+// The choice of one token by one warp: logits z [E + groups.count] (shared memory; the entries behind the
+// logits are scratch), the bias already in.
 __device__ __forceinline__ void router_choose(float* z, int E, int top, int renormalize, int score_mode, int* my_ids, float* my_w,
-                                              int lane, const float* __restrict__ correction) {
+                                              int lane, const float* __restrict__ correction, const RouterGroups& groups) {
   if (score_mode == ROUTER_SCORE_SOFTMAX_ALL) {
     // z becomes the softmax over all experts; the choice below then runs over z + correction
     float mx = -INFINITY, sum = 0.f;
@@ -44,6 +54,23 @@ __device__ __forceinline__ void router_choose(float* z, int E, int top, int reno
     for (int e = lane; e < E; e += 32) sum += expf(z[e] - mx);
     sum = ts_warp_sum(sum);
     for (int e = lane; e < E; e += 32) z[e] = expf(z[e] - mx) / sum;
+    __syncwarp();
+  }
+  if (groups.count > 1 && groups.keep < groups.count) {
+    const int n = E / groups.count;
+    float* best_of = z + E;
+    for (int g = lane; g < groups.count; g += 32) {
+      float m = -INFINITY;
+      for (int e = g * n; e < (g + 1) * n; ++e) m = fmaxf(m, z[e] + (correction ? correction[e] : 0.f));
+      best_of[g] = m;
+    }
+    __syncwarp();
+    for (int g = lane; g < groups.count; g += 32) {
+      int before = 0;  // groups that are kept ahead of this one (the lower index wins a tie)
+      for (int j = 0; j < groups.count; ++j) before += best_of[j] > best_of[g] || (best_of[j] == best_of[g] && j < g);
+      if (before >= groups.keep)
+        for (int e = g * n; e < (g + 1) * n; ++e) z[e] = -INFINITY;  // never the largest of what is left
+    }
     __syncwarp();
   }
   float total = 0.f, first = 0.f;
@@ -78,30 +105,42 @@ __device__ __forceinline__ void router_choose(float* z, int E, int top, int reno
     }
     __syncwarp();
   }
-  if ((renormalize || score_mode == ROUTER_SCORE_SOFTMAX_CHOSEN) && lane == 0)
-    for (int k = 0; k < top; ++k) my_w[k] /= total;
+  if (lane == 0) {
+    if (renormalize || score_mode == ROUTER_SCORE_SOFTMAX_CHOSEN)
+      for (int k = 0; k < top; ++k) my_w[k] /= total + 1e-20f;
+    if (groups.scale != 1.f)
+      for (int k = 0; k < top; ++k) my_w[k] *= groups.scale;
+  }
 }
 
 __global__ void router_topk_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int T, int E, int top, int renormalize,
-                                   int score_mode, int* __restrict__ ids, float* __restrict__ weights, const float* __restrict__ correction) {
+                                   int score_mode, int* __restrict__ ids, float* __restrict__ weights, const float* __restrict__ correction, RouterGroups groups) {
   ts_pdl_prologue();
-  extern __shared__ float zs[];  // [4][E]: a token's logits with the bias added
+  extern __shared__ float zs[];  // [4][E + groups]: a token's logits with the bias added, and the choice's scratch
   const int w = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int warp = blockIdx.x * (blockDim.x >> 5) + w;
   if (warp >= T) return;
-  float* z = zs + (size_t)w * E;
+  float* z = zs + (size_t)w * (E + groups.count);
   for (int e = lane; e < E; e += 32) z[e] = logits[(size_t)warp * E + e] + (bias ? bias[e] : 0.f);
   __syncwarp();
-  router_choose(z, E, top, renormalize, score_mode, ids + (size_t)warp * top, weights + (size_t)warp * top, lane, correction);
+  router_choose(z, E, top, renormalize, score_mode, ids + (size_t)warp * top, weights + (size_t)warp * top, lane, correction, groups);
+}
+
+// Whether every choice of `top` experts finds as many inside the kept groups.
+static inline bool router_groups_fit(int E, int top, int count, int keep) {
+  if (count <= 1) return count >= 0;
+  return E % count == 0 && keep >= 1 && keep <= count && top <= keep * (E / count);
 }
 
 TS_EXPORT int ts_router_topk(const float* logits, const float* bias, int T, int E, int top, int renormalize, int score_mode, int* ids,
-                             float* weights, const float* correction, void* stream) {
+                             float* weights, const float* correction, int group_count, int group_keep, float scale, void* stream) {
   if (T <= 0) return 0;
-  if (E <= 0 || top <= 0 || top > E) return TS_ERR_BAD_ARGUMENT;
-  if ((size_t)4 * E * sizeof(float) > 48 * 1024) return TS_ERR_UNSUPPORTED_SIZE;
-  return ts_launch(router_topk_kernel, dim3((T + 3) / 4), dim3(128), (size_t)4 * E * sizeof(float), (cudaStream_t)stream, logits, bias, T, E,
-                   top, renormalize, score_mode, ids, weights, correction);
+  if (E <= 0 || top <= 0 || top > E || !router_groups_fit(E, top, group_count, group_keep)) return TS_ERR_BAD_ARGUMENT;
+  const RouterGroups groups = {group_count, group_keep, scale};
+  const size_t smem = (size_t)4 * (E + group_count) * sizeof(float);
+  if (smem > 48 * 1024) return TS_ERR_UNSUPPORTED_SIZE;
+  return ts_launch(router_topk_kernel, dim3((T + 3) / 4), dim3(128), smem, (cudaStream_t)stream, logits, bias, T, E,
+                   top, renormalize, score_mode, ids, weights, correction, groups);
 }
 
 // One block: counts per expert, their prefix sums, then every pair takes the next place of its expert.
@@ -358,11 +397,12 @@ template <typename TX>
 __global__ void __launch_bounds__(256) router_kernel(const TX* __restrict__ x, const float* __restrict__ router,
                                                      const float* __restrict__ bias, int T, int W, int E, int top, int renormalize,
                                                      int score_mode, int rt, int* __restrict__ ids, float* __restrict__ weights,
-                                                     const float* __restrict__ correction) {
+                                                     const float* __restrict__ correction, RouterGroups groups) {
   ts_pdl_prologue();
   extern __shared__ float rs[];
   float* xs = rs;                    // [rt][W]
-  float* logits = rs + (size_t)rt * W;  // [rt][E]
+  const int Z = E + groups.count;
+  float* logits = rs + (size_t)rt * W;  // [rt][E + groups]
   const int t0 = blockIdx.x * rt;
   const int nt = min(rt, T - t0);
   for (int i = threadIdx.x; i < nt * W; i += blockDim.x) xs[i] = ts_to_float(x[(size_t)t0 * W + i]);
@@ -397,24 +437,27 @@ __global__ void __launch_bounds__(256) router_kernel(const TX* __restrict__ x, c
 #pragma unroll
     for (int j = 0; j < ROUTER_MAX_TOKENS; ++j) {
       const float v = ts_warp_sum(acc[j]);
-      if (lane == 0 && j < nt) logits[(size_t)j * E + e] = v + (bias ? bias[e] : 0.f);
+      if (lane == 0 && j < nt) logits[(size_t)j * Z + e] = v + (bias ? bias[e] : 0.f);
     }
   }
   __syncthreads();
   if (warp >= nt) return;
-  router_choose(logits + (size_t)warp * E, E, top, renormalize, score_mode, ids + (size_t)(t0 + warp) * top,
-                weights + (size_t)(t0 + warp) * top, lane, correction);
+  router_choose(logits + (size_t)warp * Z, E, top, renormalize, score_mode, ids + (size_t)(t0 + warp) * top,
+                weights + (size_t)(t0 + warp) * top, lane, correction, groups);
 }
 
 TS_EXPORT int ts_router(const void* x, int x_dtype, const float* router, const float* bias, int T, int W, int E, int top, int renormalize,
-                        int score_mode, int* ids, float* weights, const float* correction, void* stream) {
+                        int score_mode, int* ids, float* weights, const float* correction, int group_count, int group_keep, float scale,
+                        void* stream) {
   if (T <= 0) return 0;
-  if (W <= 0 || E <= 0 || top <= 0 || top > E) return TS_ERR_BAD_ARGUMENT;
+  if (W <= 0 || E <= 0 || top <= 0 || top > E || !router_groups_fit(E, top, group_count, group_keep)) return TS_ERR_BAD_ARGUMENT;
+  const RouterGroups groups = {group_count, group_keep, scale};
+  const int Z = E + group_count;
   // tokens per CTA: four where there are CTAs enough for every SM several times over (a router row is
   // then read once per four tokens), fewer in steps of few tokens (more CTAs, shorter chains of loads)
   int rt = T >= 2048 ? ROUTER_MAX_TOKENS : (T >= 512 ? 2 : 1);
-  while (rt > 1 && (size_t)rt * (W + E) * sizeof(float) > 200 * 1024) rt >>= 1;
-  const size_t smem = (size_t)rt * (W + E) * sizeof(float);
+  while (rt > 1 && (size_t)rt * (W + Z) * sizeof(float) > 200 * 1024) rt >>= 1;
+  const size_t smem = (size_t)rt * (W + Z) * sizeof(float);
   if (smem > 227 * 1024) return TS_ERR_UNSUPPORTED_SIZE;
   cudaStream_t s = (cudaStream_t)stream;
   const dim3 grid((T + rt - 1) / rt);
@@ -425,7 +468,7 @@ TS_EXPORT int ts_router(const void* x, int x_dtype, const float* router, const f
       if (e != cudaSuccess) return (int)e;
       set32 = 227 * 1024;
     }
-    return ts_launch(router_kernel<float>, grid, dim3(256), smem, s, (const float*)x, router, bias, T, W, E, top, renormalize, score_mode, rt, ids, weights, correction);
+    return ts_launch(router_kernel<float>, grid, dim3(256), smem, s, (const float*)x, router, bias, T, W, E, top, renormalize, score_mode, rt, ids, weights, correction, groups);
   }
   if (x_dtype == TS_DTYPE_BF16) {
     static size_t set16 = 0;
@@ -435,7 +478,7 @@ TS_EXPORT int ts_router(const void* x, int x_dtype, const float* router, const f
       set16 = 227 * 1024;
     }
     return ts_launch(router_kernel<__nv_bfloat16>, grid, dim3(256), smem, s, (const __nv_bfloat16*)x, router, bias, T, W, E, top, renormalize,
-                     score_mode, rt, ids, weights, correction);
+                     score_mode, rt, ids, weights, correction, groups);
   }
   return TS_ERR_BAD_ARGUMENT;
 }

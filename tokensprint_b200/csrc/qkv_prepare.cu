@@ -14,11 +14,19 @@
 //               written to q_out [T, nq, D], entries d..D-1 zero.  For a key head the same, stored
 //               at the token's cache slot in k_dst [slots, nkv, D]; the value head of the same index
 //               (e entries, bias, nothing else) goes to v_dst [slots, nkv, D], entries e..D-1 zero.
+//               With weights `q_norm` / `k_norm` [d] every head is first brought to unit root mean square and
+//               multiplied by them (before the rotation; after the bias).  With `first` (rows of another
+//               layer's values of the same tokens, nkv*e wide) the stored values are
+//               (1 - share) v + share first.
 //               D >= max(d, e): a kernel compiled for heads of D entries then runs heads whose keys
 //               and values differ in width (zeros add nothing to a score and are never read back).
 //               All arithmetic is float32; inputs and outputs are in the activation type.
 // gate_rows:    y[t, h*e + i] = a[t, h, i] * sigmoid(g[t, h*e + i]) (a has rows of D >= e entries per
-//               head; g null: a plain compaction), the gate in float32.
+//               head; g null: a plain compaction), the gate in float32; per_head: one gate for a whole
+//               head, g[t, h].
+// rotate_qkv:   out[t] = [rotated q | rotated k | v] in float32 from columns of one product's result: the
+//               first `rot` entries of every head of q and k turn by the table (pairs (i, i + rot/2)), the rest
+//               and the values pass; for recurrences over rotated keys, which take float32 rows.
 #include "common.cuh"
 
 #define QP_WARPS 4
@@ -48,7 +56,8 @@ __global__ void __launch_bounds__(QP_WARPS * 32) qkv_prepare_kernel(
     const TA* __restrict__ proj, long long ld, int q_off, int k_off, int v_off, const float* __restrict__ q_bias,
     const float* __restrict__ k_bias, const float* __restrict__ v_bias, const float2* __restrict__ table, int rot, int unit_norm, float eps,
     TA* __restrict__ q_out, TA* __restrict__ k_dst, TA* __restrict__ v_dst, const int* __restrict__ slot_mapping, int T, int nq, int nkv,
-    int d, int e, int D, const int* __restrict__ positions, float qt_coef, int qt_every) {
+    int d, int e, int D, const int* __restrict__ positions, float qt_coef, int qt_every, const float* __restrict__ q_norm,
+    const float* __restrict__ k_norm, const TA* __restrict__ first, long long ld_first, float share) {
   ts_pdl_prologue();
   __shared__ float buf[QP_WARPS][QP_MAX_DIM];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -68,17 +77,30 @@ __global__ void __launch_bounds__(QP_WARPS * 32) qkv_prepare_kernel(
   if (bias != nullptr) bias += (size_t)h * d;
   const int half = rot >> 1;
   float* x = buf[warp];
+  const float* nw = is_q ? q_norm : k_norm;
+  float pre = 1.f;
+  if (nw != nullptr) {
+    float s2 = 0.f;
+    for (int i = lane; i < d; i += 32) {
+      const float u = ts_to_float(row[i]) + (bias ? bias[i] : 0.f);
+      s2 += u * u;
+    }
+    pre = 1.f / sqrtf(ts_warp_sum(s2) / (float)d + eps);
+  }
+  auto entry = [&](int i) {
+    const float u = ts_to_float(row[i]) + (bias ? bias[i] : 0.f);
+    return nw != nullptr ? u * pre * nw[i] : u;
+  };
   float ss = 0.f;
   for (int j = lane; j < half; j += 32) {
-    const float u = ts_to_float(row[j]) + (bias ? bias[j] : 0.f);
-    const float v = ts_to_float(row[j + half]) + (bias ? bias[j + half] : 0.f);
+    const float u = entry(j), v = entry(j + half);
     const float2 cs = table[(size_t)t * half + j];
     const float a = u * cs.x - v * cs.y, b = v * cs.x + u * cs.y;
     x[j] = a, x[j + half] = b;
     ss += a * a + b * b;
   }
   for (int i = rot + lane; i < d; i += 32) {
-    const float u = ts_to_float(row[i]) + (bias ? bias[i] : 0.f);
+    const float u = entry(i);
     x[i] = u;
     ss += u * u;
   }
@@ -92,14 +114,20 @@ __global__ void __launch_bounds__(QP_WARPS * 32) qkv_prepare_kernel(
     const TA* vrow = proj + (size_t)t * ld + v_off + (size_t)h * e;
     const float* vb = v_bias ? v_bias + (size_t)h * e : nullptr;
     TA* vd = v_dst + ((size_t)slot * nkv + h) * D;
-    for (int i = lane; i < D; i += 32) vd[i] = ts_from_float<TA>(i < e ? ts_to_float(vrow[i]) + (vb ? vb[i] : 0.f) : 0.f);
+    const TA* frow = first ? first + (size_t)t * ld_first + (size_t)h * e : nullptr;
+    for (int i = lane; i < D; i += 32) {
+      float v = i < e ? ts_to_float(vrow[i]) + (vb ? vb[i] : 0.f) : 0.f;
+      if (frow != nullptr && i < e) v = (1.f - share) * v + share * ts_to_float(frow[i]);
+      vd[i] = ts_from_float<TA>(v);
+    }
   }
 }
 
 TS_EXPORT int ts_qkv_prepare(const void* proj, int act_dtype, long long ld, int q_off, int k_off, int v_off, const float* q_bias,
                              const float* k_bias, const float* v_bias, const float* table, int rot, int unit_norm, float eps, void* q_out,
                              void* k_dst, void* v_dst, const int* slot_mapping, int T, int nq, int nkv, int d, int e, int D, const int* positions,
-                             float qt_coef, int qt_every, void* stream) {
+                             float qt_coef, int qt_every, const float* q_norm, const float* k_norm, const void* first, long long ld_first,
+                             float share, void* stream) {
   if (T <= 0) return 0;
   if (nq < 0 || nkv < 0 || nq + nkv <= 0 || d <= 0 || e <= 0 || D < d || D < e || rot < 0 || rot > d || (rot & 1) || (rot > 0 && table == nullptr) ||
       qt_every < 0 || (qt_every > 0 && positions == nullptr))
@@ -111,24 +139,26 @@ TS_EXPORT int ts_qkv_prepare(const void* proj, int act_dtype, long long ld, int 
   const float2* tb = reinterpret_cast<const float2*>(table);
   if (act_dtype == TS_DTYPE_F32)
     return ts_launch(qkv_prepare_kernel<float>, dim3(blocks), dim3(QP_WARPS * 32), 0, s, (const float*)proj, ld, q_off, k_off, v_off, q_bias,
-                     k_bias, v_bias, tb, rot, unit_norm, eps, (float*)q_out, (float*)k_dst, (float*)v_dst, slot_mapping, T, nq, nkv, d, e, D, positions, qt_coef, qt_every);
+                     k_bias, v_bias, tb, rot, unit_norm, eps, (float*)q_out, (float*)k_dst, (float*)v_dst, slot_mapping, T, nq, nkv, d, e, D, positions, qt_coef, qt_every, q_norm, k_norm,
+                     (const float*)first, ld_first, share);
   if (act_dtype == TS_DTYPE_BF16)
     return ts_launch(qkv_prepare_kernel<__nv_bfloat16>, dim3(blocks), dim3(QP_WARPS * 32), 0, s, (const __nv_bfloat16*)proj, ld, q_off, k_off,
                      v_off, q_bias, k_bias, v_bias, tb, rot, unit_norm, eps, (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_dst,
-                     (__nv_bfloat16*)v_dst, slot_mapping, T, nq, nkv, d, e, D, positions, qt_coef, qt_every);
+                     (__nv_bfloat16*)v_dst, slot_mapping, T, nq, nkv, d, e, D, positions, qt_coef, qt_every, q_norm, k_norm,
+                     (const __nv_bfloat16*)first, ld_first, share);
   return TS_ERR_BAD_ARGUMENT;
 }
 
 template <typename TA>
 __global__ void gate_rows_kernel(const TA* __restrict__ a, const TA* __restrict__ g, long long ld_g, TA* __restrict__ y, long long n, int H, int e,
-                                 int D) {
+                                 int D, int per_head) {
   ts_pdl_prologue();
   const int He = H * e;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
     const long long t = i / He;
     const int c = (int)(i - t * He), h = c / e, j = c - h * e;
     float v = ts_to_float(a[((size_t)t * H + h) * D + j]);
-    if (g != nullptr) v *= 1.f / (1.f + expf(-ts_to_float(g[(size_t)t * ld_g + c])));
+    if (g != nullptr) v *= 1.f / (1.f + expf(-ts_to_float(g[(size_t)t * ld_g + (per_head ? h : c)])));
     y[i] = ts_from_float<TA>(v);
   }
 }
@@ -156,20 +186,59 @@ __global__ void __launch_bounds__(128) gate_rows_vec_kernel(const __nv_bfloat16*
   }
 }
 
-TS_EXPORT int ts_gate_rows(const void* a, const void* g, long long ld_g, int act_dtype, void* y, int T, int H, int e, int D, void* stream) {
+TS_EXPORT int ts_gate_rows(const void* a, const void* g, long long ld_g, int act_dtype, void* y, int T, int H, int e, int D, int per_head, void* stream) {
   if (T <= 0) return 0;
   if (H <= 0 || e <= 0 || D < e) return TS_ERR_BAD_ARGUMENT;
   const long long n = (long long)T * H * e;
   const unsigned blocks = (unsigned)min((n + 255) / 256, (long long)148 * 16);
   cudaStream_t s = (cudaStream_t)stream;
   const int He = H * e;
-  if (act_dtype == TS_DTYPE_BF16 && g != nullptr && D == e && He % 8 == 0 && ld_g % 8 == 0 && (((uintptr_t)a | (uintptr_t)g | (uintptr_t)y) & 15) == 0)
+  if (act_dtype == TS_DTYPE_BF16 && g != nullptr && !per_head && D == e && He % 8 == 0 && ld_g % 8 == 0 && (((uintptr_t)a | (uintptr_t)g | (uintptr_t)y) & 15) == 0)
     return ts_launch(gate_rows_vec_kernel, dim3((unsigned)((He / 8 + 127) / 128), (unsigned)min(T, 65535)), dim3(128), 0, s, (const __nv_bfloat16*)a,
                      (const __nv_bfloat16*)g, ld_g, (__nv_bfloat16*)y, T, He);
   if (act_dtype == TS_DTYPE_F32)
-    return ts_launch(gate_rows_kernel<float>, dim3(blocks), dim3(256), 0, s, (const float*)a, (const float*)g, ld_g, (float*)y, n, H, e, D);
+    return ts_launch(gate_rows_kernel<float>, dim3(blocks), dim3(256), 0, s, (const float*)a, (const float*)g, ld_g, (float*)y, n, H, e, D, per_head);
   if (act_dtype == TS_DTYPE_BF16)
     return ts_launch(gate_rows_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, s, (const __nv_bfloat16*)a, (const __nv_bfloat16*)g, ld_g,
-                     (__nv_bfloat16*)y, n, H, e, D);
+                     (__nv_bfloat16*)y, n, H, e, D, per_head);
+  return TS_ERR_BAD_ARGUMENT;
+}
+
+// One block per token; a thread takes entries of the row [q | k | v] one block width apart.
+template <typename TA>
+__global__ void __launch_bounds__(256) rotate_qkv_kernel(const TA* __restrict__ proj, long long ld, int q_off, int k_off, int v_off,
+                                                         const float2* __restrict__ table, int half, float* __restrict__ out, int Hd, int d, int He) {
+  ts_pdl_prologue();
+  const int t = blockIdx.x;
+  const TA* row = proj + (size_t)t * ld;
+  float* o = out + (size_t)t * (2 * Hd + He);
+  const float2* cs_row = table + (size_t)t * half;
+  for (int i = threadIdx.x; i < Hd; i += blockDim.x) {
+    const int c = i % d;
+    float q = ts_to_float(row[q_off + i]), k = ts_to_float(row[k_off + i]);
+    if (c < 2 * half) {
+      const bool low = c < half;
+      const int other = low ? i + half : i - half;
+      const float2 cs = cs_row[low ? c : c - half];
+      const float sn = low ? -cs.y : cs.y;
+      q = q * cs.x + ts_to_float(row[q_off + other]) * sn;
+      k = k * cs.x + ts_to_float(row[k_off + other]) * sn;
+    }
+    o[i] = q, o[Hd + i] = k;
+  }
+  for (int i = threadIdx.x; i < He; i += blockDim.x) o[2 * Hd + i] = ts_to_float(row[v_off + i]);
+}
+
+TS_EXPORT int ts_rotate_qkv(const void* proj, int act_dtype, long long ld, int q_off, int k_off, int v_off, const float* table, int rot, float* out,
+                            int T, int H, int d, int e, void* stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || d <= 0 || e <= 0 || rot < 0 || rot > d || (rot & 1) || (rot > 0 && table == nullptr)) return TS_ERR_BAD_ARGUMENT;
+  cudaStream_t s = (cudaStream_t)stream;
+  const float2* tb = reinterpret_cast<const float2*>(table);
+  if (act_dtype == TS_DTYPE_F32)
+    return ts_launch(rotate_qkv_kernel<float>, dim3(T), dim3(256), 0, s, (const float*)proj, ld, q_off, k_off, v_off, tb, rot / 2, out, H * d, d, H * e);
+  if (act_dtype == TS_DTYPE_BF16)
+    return ts_launch(rotate_qkv_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, s, (const __nv_bfloat16*)proj, ld, q_off, k_off, v_off, tb, rot / 2, out,
+                     H * d, d, H * e);
   return TS_ERR_BAD_ARGUMENT;
 }

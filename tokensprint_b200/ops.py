@@ -53,9 +53,10 @@ _SIGNATURES = {
     "ts_gelu_tanh": [_c_void_p, _c_void_p, _c_int, _c_ll, _c_void_p],
     "ts_capped_glu": [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_float, _c_void_p],
     "ts_gelu_gate_rows": [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_ll, _c_int, _c_int, _c_void_p],
-    "ts_router_topk": [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p],
+    "ts_router_topk": [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_float,
+                       _c_void_p],
     "ts_router": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p,
-                  _c_void_p],
+                  _c_int, _c_int, _c_float, _c_void_p],
     "ts_moe_gate_up_mma": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int,
                            _c_int, _c_int, _c_float, _c_float, _c_int, _c_int, _c_void_p],
     "ts_moe_down_mma": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
@@ -68,7 +69,7 @@ _SIGNATURES = {
     "ts_gla_decay": [_c_void_p, _c_ll, _c_int, _c_void_p, _c_float, _c_void_p, _c_int, _c_int, _c_void_p],
     "ts_gla_scan": [_c_void_p, _c_void_p, _c_void_p, _c_ll, _c_int, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                     _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
-    "ts_gla_norm_gate": [_c_void_p, _c_void_p, _c_ll, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_void_p],
+    "ts_gla_norm_gate": [_c_void_p, _c_void_p, _c_ll, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p],
     "ts_branch_norm_add": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_float,
                            _c_void_p],
     "ts_stream_add": [_c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p],
@@ -780,23 +781,28 @@ def gla_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor,
         launch_count += 1  # the recurrence ran as two kernels
 
 
-def gla_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, num_heads: int, value_dim: int, eps: float) -> None:
-    """out[t, h] = o[t, h] * rsqrt(mean(o[t, h]^2) + eps) * weight * silu(gate[t, h]) per head of `value_dim`
-    entries.  o [T, H*e] float32; gate [T, H*e] (any row stride) and out [T, H*e] in the compute type;
-    weight [e] float32, the same for every head."""
+def gla_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.Tensor], out: torch.Tensor, num_heads: int, value_dim: int,
+                  eps: float, activation: str = "silu") -> None:
+    """out[t, h] = o[t, h] * rsqrt(mean(o[t, h]^2) + eps) * weight * act(gate[t, h]) per head of `value_dim`
+    entries.  o [T, H*e] float32; gate [T, H*e] (any row stride) and out [T, H*e] in the compute type (the gate
+    may also be float32); weight [e] float32, the same for every head, or None; act: "silu" or "sigmoid"."""
     flush_gemm_chain()
     H, e = int(num_heads), int(value_dim)
+    if activation not in ("silu", "sigmoid"):
+        raise KernelError(f"gla_norm_gate: the gate passes through silu or the sigmoid, not {activation!r}")
     _cuda_contig("o", o, torch.float32)
-    _cuda_contig("weight", weight, torch.float32)
+    if weight is not None:
+        _cuda_contig("weight", weight, torch.float32)
     _cuda_contig("out", out)
     T = o.shape[0]
-    if not gate.is_cuda or gate.dim() != 2 or gate.stride(1) != 1 or tuple(gate.shape) != (T, H * e) or gate.dtype != out.dtype:
-        raise KernelError(f"gla_norm_gate: gate must be a CUDA matrix [{T}, {H * e}] of {out.dtype}, got {tuple(gate.shape)} {gate.dtype}")
-    if o.shape != (T, H * e) or out.shape != (T, H * e) or weight.numel() != e:
+    if gate.dtype != torch.float32 and gate.dtype != out.dtype:
+        raise KernelError(f"gla_norm_gate: the gate must be float32 or {out.dtype}, got {gate.dtype}")
+    _matrix_view("gla_norm_gate: gate", gate, T, H * e)
+    if o.shape != (T, H * e) or out.shape != (T, H * e) or (weight is not None and weight.numel() != e):
         raise KernelError("gla_norm_gate: shapes disagree")
-    _check("gla_norm_gate", _fn("ts_gla_norm_gate")(o.data_ptr(), gate.data_ptr(), gate.stride(0), _act_code("out", out), weight.data_ptr(),
-                                                    out.data_ptr(), T, H, e, float(eps), _stream()))
-
+    _check("gla_norm_gate", _fn("ts_gla_norm_gate")(o.data_ptr(), gate.data_ptr(), gate.stride(0), _act_code("gate", gate), _act_code("out", out),
+                                                    _ptr(weight), out.data_ptr(), T, H, e, float(eps), 1 if activation == "sigmoid" else 0,
+                                                    _stream()))
 
 
 # ---------------------------------------------------------------------------
@@ -805,7 +811,7 @@ def gla_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, out
 
 _SIGNATURES.update({
     "ts_linear_scan": [_c_void_p, _c_void_p, _c_void_p, _c_ll, _c_int, _c_void_p, _c_int, _c_void_p, _c_float, _c_void_p, _c_ll, _c_void_p,
-                       _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
+                       _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p],
     "ts_rows_dot_f32": [_c_void_p, _c_int, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
     "ts_mlstm_gate_scan": [_c_void_p, _c_void_p, _c_float, _c_void_p, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p],
     "ts_mlstm_norm_gate": [_c_void_p, _c_void_p, _c_void_p, _c_ll, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_void_p],
@@ -818,13 +824,16 @@ _SIGNATURES.update({
     "ts_rope_table": [_c_void_p, _c_void_p, _c_float, _c_int, _c_int, _c_void_p, _c_void_p],
     "ts_qkv_prepare": [_c_void_p, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_float,
                        _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_float, _c_int,
-                       _c_void_p],
+                       _c_void_p, _c_void_p, _c_void_p, _c_ll, _c_float, _c_void_p],
+    "ts_rotate_qkv": [_c_void_p, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "ts_softcap_rows": [_c_void_p, _c_ll, _c_float, _c_void_p],
     "ts_causal_conv": [_c_void_p, _c_int, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                        _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_void_p],
-    "ts_delta_scan": [_c_void_p, _c_ll, _c_int, _c_int, _c_int, _c_void_p, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_ll, _c_void_p, _c_void_p,
-                      _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_void_p],
-    "ts_gate_rows": [_c_void_p, _c_void_p, _c_ll, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+    "ts_delta_scan": [_c_void_p, _c_ll, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_ll, _c_void_p, _c_ll, _c_int, _c_int, _c_void_p, _c_void_p,
+                      _c_void_p, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int,
+                      _c_void_p],
+    "ts_channel_decay": [_c_void_p, _c_ll, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
+    "ts_gate_rows": [_c_void_p, _c_void_p, _c_ll, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "ts_weighted_sum": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_float, _c_float, _c_float, _c_float, _c_int, _c_void_p, _c_int, _c_ll,
                         _c_void_p],
 })
@@ -838,16 +847,19 @@ def _matrix_view(name: str, t: torch.Tensor, rows: int, cols: int, dtype: Option
 
 def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, kscale: Optional[torch.Tensor], q_scale: float,
                 state: torch.Tensor, state_slots: torch.Tensor, cu_seqlens: torch.Tensor, out: torch.Tensor, num_seqs: int, num_heads: int,
-                groups: int, key_dim: int, value_dim: int, normaliser: bool = False, max_seqlen: Optional[int] = None) -> None:
+                groups: int, key_dim: int, value_dim: int, normaliser: bool = False, max_seqlen: Optional[int] = None,
+                rotation: Optional[torch.Tensor] = None) -> None:
     """S_t = a_t S_(t-1) + (b_t k_t) v_t^T,  out_t = S_t^T (q_t * q_scale), per head, over the step's tokens
-    sequence by sequence, with one decay a_t per (token, head).
+    sequence by sequence, with one decay a_t per (token, head), or (decay [H]) one constant per head.
 
     q, k [T, groups*d] (head h reads group h // (H // groups)) and v [T, H*e]: views with one common
     row stride, float32 or bfloat16 (all three alike); decay [T, H] and kscale [T, H] (or None) float32.
     state [slots, n] float32 with n >= H*d*e': a request's [H, d, e'] block stands at the start of its
     row, e' = e + 1 with `normaliser` (the extra column is fed the value 1 in every token, so it holds
     the sum of the decayed b_t k_t, and its read-out arrives as column e of out), else e' = e.
-    out [T, H*e'] float32.  Long portions run in segments side by side as in gla_scan."""
+    out [T, H*e'] float32.  Long portions run in segments side by side as in gla_scan.
+    `rotation` [T, r/2, 2] float32 (rope_table), in steps of one token per sequence only (max_seqlen = 1): the first r
+    entries of every q and k head turn by it as they are read; longer portions bring rotated rows (rotate_qkv)."""
     flush_gemm_chain()
     H, G, d, e = int(num_heads), int(groups), int(key_dim), int(value_dim)
     ee = e + 1 if normaliser else e
@@ -864,9 +876,16 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.
     _cuda_contig("decay", decay, torch.float32)
     if kscale is not None:
         _cuda_contig("kscale", kscale, torch.float32)
-    for name, t in (("decay", decay), ("kscale", kscale)):
-        if t is not None and tuple(t.shape) != (T, H):
-            raise KernelError(f"linear_scan: {name} must be [{T}, {H}], got {tuple(t.shape)}")
+    constant = decay.dim() == 1
+    for name, t, shape in (("decay", decay, (H,) if constant else (T, H)), ("kscale", kscale, (T, H))):
+        if t is not None and tuple(t.shape) != shape:
+            raise KernelError(f"linear_scan: {name} must be {list(shape)}, got {tuple(t.shape)}")
+    half = 0
+    if rotation is not None:
+        _cuda_contig("rotation", rotation, torch.float32)
+        half = rotation.shape[1]
+        if max_seqlen != 1 or rotation.dim() != 3 or rotation.shape[0] < T or rotation.shape[2] != 2 or 2 * half > d:
+            raise KernelError(f"linear_scan: a rotation is [T, r/2, 2] with r <= {d} and comes in steps of one token, got {tuple(rotation.shape)}")
     _cuda_contig("state_slots", state_slots, torch.int32)
     _cuda_contig("cu_seqlens", cu_seqlens, torch.int32)
     _cuda_contig("out", out, torch.float32)
@@ -884,9 +903,9 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.
         need = int(num_seqs) * segs * H * d * ee + int(num_seqs) * segs * H * d + int(num_seqs) * H * d * ee
         scratch = torch.empty(need, device=q.device, dtype=torch.float32)
     _check("linear_scan", _fn("ts_linear_scan")(
-        q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), _act_code("q", q), decay.data_ptr(), 1, _ptr(kscale), float(q_scale),
-        state.data_ptr(), state.stride(0), state_slots.data_ptr(), cu_seqlens.data_ptr(), out.data_ptr(), int(num_seqs), H, G, d, e, ee,
-        segs, seg_len, _ptr(scratch), _stream()))
+        q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), _act_code("q", q), decay.data_ptr(), 2 if constant else 1, _ptr(kscale),
+        float(q_scale), state.data_ptr(), state.stride(0), state_slots.data_ptr(), cu_seqlens.data_ptr(), out.data_ptr(), int(num_seqs), H, G, d, e,
+        ee, segs, seg_len, _ptr(scratch), _ptr(rotation), half, _stream()))
     if segs > 1:
         global launch_count
         launch_count += 1  # the recurrence ran as two kernels
@@ -1154,16 +1173,32 @@ DELTA_MAX_KEY_DIM = 1024
 DELTA_LANES = int(_os.environ.get("TS_DELTA_LANES", "0"))
 
 
-def delta_scan(x: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
-               state: torch.Tensor, state_slots: torch.Tensor, cu_seqlens: torch.Tensor, out: torch.Tensor, num_seqs: int, num_heads: int,
-               num_qk_heads: int, key_dim: int, value_dim: int, q_scale: float, unit_eps: float) -> None:
+def channel_decay(z: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, num_heads: int, key_dim: int) -> None:
+    """z <- exp(-exp(a_log_h) * softplus(z + dt_bias)) in place, float32: a decay per (token, head, key channel).
+    z [T, H*d] (any row stride), a_log [H], dt_bias [H*d]."""
+    flush_gemm_chain()
+    H, d = int(num_heads), int(key_dim)
+    T = z.shape[0]
+    _matrix_view("channel_decay: z", z, T, H * d, torch.float32)
+    _cuda_contig("a_log", a_log, torch.float32)
+    _cuda_contig("dt_bias", dt_bias, torch.float32)
+    if a_log.numel() != H or dt_bias.numel() != H * d:
+        raise KernelError("channel_decay: a_log needs one entry per head, dt_bias one per head and key channel")
+    _check("channel_decay", _fn("ts_channel_decay")(z.data_ptr(), z.stride(0), a_log.data_ptr(), dt_bias.data_ptr(), T, H, d, _stream()))
+
+
+def delta_scan(x: torch.Tensor, q_off: int, k_off: int, v_off: int, beta: torch.Tensor, decay: torch.Tensor, a_log: Optional[torch.Tensor],
+               dt_bias: Optional[torch.Tensor], state: torch.Tensor, state_slots: torch.Tensor, cu_seqlens: torch.Tensor, out: torch.Tensor,
+               num_seqs: int, num_heads: int, num_qk_heads: int, key_dim: int, value_dim: int, q_scale: float, unit_eps: float) -> None:
     """The gated delta rule over the tokens of every sequence, in order (csrc/delta_rule.cu).  x [T, n]
     float32 holds q (columns q_off.., num_qk_heads * key_dim), k (k_off..) and v (v_off.., num_heads *
     value_dim); q and k are brought to unit length per head here and q is multiplied by q_scale.
-    gates [T, 2 * heads] float32: the raw write-strength rows, then the raw decay rows (beta = sigmoid,
-    decay = exp(-exp(a_log) * softplus(raw + dt_bias))).  state [slots, >= heads * value_dim * key_dim]
-    float32 (a view with a row stride is fine), one head after the other, value column by value column;
-    out [T, heads * value_dim] float32."""
+    beta [T, heads] float32 or bfloat16: the raw write strengths (the sigmoid is taken here).  decay float32,
+    [T, heads] (one per head) or [T, heads * key_dim] (one per key channel): with a_log and dt_bias (one entry
+    per column of decay) the raw rows, of which exp(-exp(a_log) * softplus(raw + dt_bias)) is taken here;
+    with None for both the decays themselves.  beta and decay may be column ranges of wider matrices.
+    state [slots, >= heads * value_dim * key_dim] float32 (a view with a row stride is fine), one head after the
+    other, value column by value column; out [T, heads * value_dim] float32."""
     flush_gemm_chain()
     H, G, d, e = int(num_heads), int(num_qk_heads), int(key_dim), int(value_dim)
     T = x.shape[0]
@@ -1171,20 +1206,28 @@ def delta_scan(x: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: torch
         raise KernelError("delta_scan: x must be a float32 CUDA matrix with unit inner stride")
     if max(q_off, k_off) + G * d > x.shape[1] or v_off + H * e > x.shape[1]:
         raise KernelError("delta_scan: the column ranges do not fit x")
-    _matrix_view("delta_scan: gates", gates, T, 2 * H, torch.float32)
-    _cuda_contig("a_log", a_log, torch.float32)
-    _cuda_contig("dt_bias", dt_bias, torch.float32)
+    _matrix_view("delta_scan: beta", beta, T, H)
+    per_channel = decay.dim() == 2 and decay.shape[1] == H * d and d > 1
+    _matrix_view("delta_scan: decay", decay, T, H * d if per_channel else H, torch.float32)
+    if (a_log is None) != (dt_bias is None):
+        raise KernelError("delta_scan: a_log and dt_bias come together (raw decay rows) or not at all (decays)")
+    if a_log is not None:
+        _cuda_contig("a_log", a_log, torch.float32)
+        _cuda_contig("dt_bias", dt_bias, torch.float32)
+        if a_log.numel() != H or dt_bias.numel() != decay.shape[1]:
+            raise KernelError("delta_scan: a_log needs one entry per head, dt_bias one per column of the decay rows")
     _cuda_contig("out", out, torch.float32)
-    if a_log.numel() != H or dt_bias.numel() != H or out.shape != (T, H * e):
-        raise KernelError("delta_scan: a_log and dt_bias need one entry per head, out must be [T, heads * value_dim]")
+    if out.shape != (T, H * e):
+        raise KernelError("delta_scan: out must be [T, heads * value_dim]")
     if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < H * d * e:
         raise KernelError(f"delta_scan: the state must be float32 [slots, >= {H * d * e}], got {tuple(state.shape)}")
     if d > DELTA_MAX_KEY_DIM or H % G:
         raise KernelError(f"delta_scan: key_dim at most {DELTA_MAX_KEY_DIM}, heads a multiple of the q/k heads")
     _check("delta_scan", _fn("ts_delta_scan")(
-        x.data_ptr(), x.stride(0), int(q_off), int(k_off), int(v_off), gates.data_ptr(), gates.stride(0), a_log.data_ptr(), dt_bias.data_ptr(),
-        state.data_ptr(), state.stride(0), state_slots.data_ptr(), cu_seqlens.data_ptr(), out.data_ptr(), int(num_seqs), H, G, d, e,
-        float(q_scale), float(unit_eps), DELTA_LANES, _stream()))
+        x.data_ptr(), x.stride(0), int(q_off), int(k_off), int(v_off), beta.data_ptr(), _act_code("beta", beta), beta.stride(0), decay.data_ptr(),
+        decay.stride(0), 1 if per_channel else 0, 0 if a_log is None else 1, _ptr(a_log), _ptr(dt_bias), state.data_ptr(), state.stride(0),
+        state_slots.data_ptr(), cu_seqlens.data_ptr(), out.data_ptr(), int(num_seqs), H, G, d, e, float(q_scale), float(unit_eps), DELTA_LANES,
+        _stream()))
 
 
 WEIGHTED_SUM_MAX_INPUTS = 4
@@ -1231,7 +1274,8 @@ def qkv_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_bias: 
                 v_bias: Optional[torch.Tensor], table: Optional[torch.Tensor], unit_norm: bool, eps: float, q_out: torch.Tensor,
                 k_dst: Optional[torch.Tensor], v_dst: Optional[torch.Tensor], slot_mapping: Optional[torch.Tensor], num_heads: int,
                 num_kv_heads: int, key_dim: int, value_dim: int, padded_dim: int, positions: Optional[torch.Tensor] = None,
-                query_temperature: Optional[tuple[float, int]] = None) -> None:
+                query_temperature: Optional[tuple[float, int]] = None, q_norm: Optional[torch.Tensor] = None,
+                k_norm: Optional[torch.Tensor] = None, first_values: Optional[torch.Tensor] = None, value_share: float = 0.0) -> None:
     """Queries, keys and values of a step out of one projection's result `proj` [T, n] (columns q_off..,
     k_off.., v_off..): biases [heads*dim] float32 (or None), rotation of the first 2*table.shape[1]
     entries of every q and k head by the table's (cos, sin) (rope_table; None: no rotation), then with
@@ -1239,7 +1283,10 @@ def qkv_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_bias: 
     k_dst / v_dst [slots, nkv, D] at slot_mapping[t] (None: row t; a negative slot: not kept), padded with
     zeros from their own width to D = padded_dim.  k_dst None: only the queries are made.
     query_temperature = (coef, every) with the tokens' positions: query heads are multiplied by
-    1 + coef * ln(floor((position + 1) / every) + 1)."""
+    1 + coef * ln(floor((position + 1) / every) + 1).
+    q_norm / k_norm [key_dim] float32: every q / k head is brought to unit root mean square (`eps` under the root)
+    and multiplied by the weight, before the rotation.  first_values [T, nkv*e] (any row stride): the stored values
+    are (1 - value_share) * v + value_share * first_values."""
     flush_gemm_chain()
     qt_coef, qt_every = (0.0, 0) if query_temperature is None else (float(query_temperature[0]), int(query_temperature[1]))
     if qt_every:
@@ -1260,6 +1307,13 @@ def qkv_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_bias: 
     for name, t in (("q_bias", q_bias), ("k_bias", k_bias), ("v_bias", v_bias)):
         if t is not None:
             _cuda_contig(name, t, torch.float32)
+    for name, t in (("q_norm", q_norm), ("k_norm", k_norm)):
+        if t is not None:
+            _cuda_contig(name, t, torch.float32)
+            if t.numel() != d:
+                raise KernelError(f"qkv_prepare: {name} must have one entry per entry of a head ({d}), got {tuple(t.shape)}")
+    if first_values is not None:
+        _matrix_view("qkv_prepare: first_values", first_values, T, nkv * e, proj.dtype)
     rot = 0
     if table is not None:
         _cuda_contig("table", table, torch.float32)
@@ -1279,12 +1333,37 @@ def qkv_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_bias: 
     _check("qkv_prepare", _fn("ts_qkv_prepare")(
         proj.data_ptr(), _act_code("proj", proj), proj.stride(0), int(q_off), int(k_off), int(v_off), _ptr(q_bias), _ptr(k_bias), _ptr(v_bias),
         _ptr(table), rot, 1 if unit_norm else 0, float(eps), q_out.data_ptr(), _ptr(k_dst), _ptr(v_dst), _ptr(slot_mapping), T, nq, kv_heads,
-        d, e, D, _ptr(positions) if qt_every else None, qt_coef, qt_every, _stream()))
+        d, e, D, _ptr(positions) if qt_every else None, qt_coef, qt_every, _ptr(q_norm), _ptr(k_norm), _ptr(first_values),
+        0 if first_values is None else first_values.stride(0), float(value_share), _stream()))
 
 
-def gate_rows(a: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, num_heads: int, value_dim: int, padded_dim: int) -> None:
+def rotate_qkv(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, table: Optional[torch.Tensor], num_heads: int, key_dim: int,
+               value_dim: int) -> torch.Tensor:
+    """[T, 2*H*d + H*e] float32: the q, k (rotated by the table over the first 2*table.shape[1] entries of every
+    head, pairs half a rotated width apart; None: as they are) and v columns of one projection's result."""
+    flush_gemm_chain()
+    H, d, e = int(num_heads), int(key_dim), int(value_dim)
+    if not proj.is_cuda or proj.dim() != 2 or proj.stride(1) != 1:
+        raise KernelError("rotate_qkv: proj must be a CUDA matrix with unit inner stride")
+    T = proj.shape[0]
+    if max(q_off, k_off) + H * d > proj.shape[1] or v_off + H * e > proj.shape[1]:
+        raise KernelError("rotate_qkv: the column ranges do not fit proj")
+    rot = 0
+    if table is not None:
+        _cuda_contig("table", table, torch.float32)
+        rot = 2 * table.shape[1]
+        if table.dim() != 3 or table.shape[0] < T or table.shape[2] != 2 or rot > d:
+            raise KernelError(f"rotate_qkv: the table must be [T, rot/2, 2] with rot <= {d}, got {tuple(table.shape)}")
+    out = torch.empty((T, 2 * H * d + H * e), device=proj.device, dtype=torch.float32)
+    _check("rotate_qkv", _fn("ts_rotate_qkv")(proj.data_ptr(), _act_code("proj", proj), proj.stride(0), int(q_off), int(k_off), int(v_off),
+                                              _ptr(table), rot, out.data_ptr(), T, H, d, e, _stream()))
+    return out
+
+
+def gate_rows(a: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, num_heads: int, value_dim: int, padded_dim: int,
+              per_head: bool = False) -> None:
     """out[t, h*e + i] = a[t, h, i] * sigmoid(gate[t, h*e + i]); a [T, H, D] with D >= e (the entries
-    beyond e are dropped); gate None: the compaction alone."""
+    beyond e are dropped); gate None: the compaction alone; per_head: gate [T, H], one number for a whole head."""
     H, e, D = int(num_heads), int(value_dim), int(padded_dim)
     _cuda_contig("a", a)
     _cuda_contig("out", out, a.dtype)
@@ -1292,9 +1371,9 @@ def gate_rows(a: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, 
     if a.numel() != T * H * D or out.shape != (T, H * e):
         raise KernelError("gate_rows: shapes disagree")
     if gate is not None:
-        _matrix_view("gate_rows: gate", gate, T, H * e, a.dtype)
+        _matrix_view("gate_rows: gate", gate, T, H if per_head else H * e, a.dtype)
     _check("gate_rows", _fn("ts_gate_rows")(a.data_ptr(), _ptr(gate), 0 if gate is None else gate.stride(0), _act_code("a", a), out.data_ptr(),
-                                            T, H, e, D, _stream()))
+                                            T, H, e, D, 1 if per_head else 0, _stream()))
 
 
 ROTARY_PAIRINGS = {"half": 0, "neighbours": 1}
@@ -1453,12 +1532,15 @@ def _router_bias(name: str, bias: Optional[torch.Tensor], E: int) -> Optional[in
 
 
 def router_topk(logits: torch.Tensor, top: int, renormalize: bool, ids: torch.Tensor, weights: torch.Tensor,
-                bias: Optional[torch.Tensor] = None, score: str = "sigmoid", correction: Optional[torch.Tensor] = None) -> None:
+                bias: Optional[torch.Tensor] = None, score: str = "sigmoid", correction: Optional[torch.Tensor] = None,
+                groups: Optional[tuple[int, int]] = None, scale: float = 1.0) -> None:
     """Per row of float32 logits [T, E] (+ bias [E], if given): the `top` experts with the largest
     logits into ids [T, top] i32 and their weights into weights [T, top] f32.  score "sigmoid": the
     weights are sigmoid(logit) (divided by their sum if `renormalize`); "softmax_chosen": the softmax
     over the chosen logits alone; "softmax_all": the scores are the softmax over all E logits, the
-    `top` largest of score + correction [E] are chosen, and the weights are the scores themselves."""
+    `top` largest of score + correction [E] are chosen, and the weights are the scores themselves (divided by
+    their sum if `renormalize`).  groups (count, keep): experts form `count` equal groups of neighbours, and only those
+    of the `keep` groups whose best member is largest may be chosen.  scale: a constant on all weights."""
     flush_gemm_chain()
     _cuda_contig("logits", logits, torch.float32)
     _cuda_contig("ids", ids, torch.int32)
@@ -1468,7 +1550,17 @@ def router_topk(logits: torch.Tensor, top: int, renormalize: bool, ids: torch.Te
         raise KernelError(f"router_topk: top {top} of {E} experts, ids {tuple(ids.shape)}, weights {tuple(weights.shape)}")
     _check("router_topk", _fn("ts_router_topk")(logits.data_ptr(), _router_bias("router_topk", bias, E), T, E, int(top),
                                                 int(bool(renormalize)), ROUTER_SCORES[score], ids.data_ptr(), weights.data_ptr(),
-                                                _router_correction("router_topk", correction, E, score), _stream()))
+                                                _router_correction("router_topk", correction, E, score),
+                                                *_router_groups("router_topk", groups, E, top), float(scale), _stream()))
+
+
+def _router_groups(name: str, groups: Optional[tuple[int, int]], E: int, top: int) -> tuple[int, int]:
+    if groups is None:
+        return 0, 0
+    count, keep = int(groups[0]), int(groups[1])
+    if count < 1 or E % count or not 1 <= keep <= count or top > keep * (E // count):
+        raise KernelError(f"{name}: {keep} of {count} groups of {E} experts cannot give {top} choices")
+    return count, keep
 
 
 def _router_correction(name: str, correction: Optional[torch.Tensor], E: int, score: str) -> Optional[int]:
@@ -1478,7 +1570,8 @@ def _router_correction(name: str, correction: Optional[torch.Tensor], E: int, sc
 
 
 def router(rows: torch.Tensor, router_weight: torch.Tensor, top: int, renormalize: bool, ids: torch.Tensor, weights: torch.Tensor,
-           bias: Optional[torch.Tensor] = None, score: str = "sigmoid", correction: Optional[torch.Tensor] = None) -> None:
+           bias: Optional[torch.Tensor] = None, score: str = "sigmoid", correction: Optional[torch.Tensor] = None,
+           groups: Optional[tuple[int, int]] = None, scale: float = 1.0) -> None:
     """Logits and choice in one kernel: rows [T, W] (float32, or bfloat16 widened on the fly) against
     router_weight [E, W] float32 with float32 sums (+ bias [E] float32, if given), then as router_topk."""
     flush_gemm_chain()
@@ -1492,7 +1585,8 @@ def router(rows: torch.Tensor, router_weight: torch.Tensor, top: int, renormaliz
         raise KernelError(f"router: rows {tuple(rows.shape)}, router {tuple(router_weight.shape)}, top {top}, ids {tuple(ids.shape)}")
     _check("router", _fn("ts_router")(rows.data_ptr(), _act_code("rows", rows), router_weight.data_ptr(), _router_bias("router", bias, E),
                                       T, W, E, int(top), int(bool(renormalize)), ROUTER_SCORES[score], ids.data_ptr(), weights.data_ptr(),
-                                      _router_correction("router", correction, E, score), _stream()))
+                                      _router_correction("router", correction, E, score), *_router_groups("router", groups, E, top),
+                                      float(scale), _stream()))
 
 
 # TS_MOE_MMA=0 (for measurements): bfloat16 expert products on CUDA cores too.
@@ -2574,6 +2668,7 @@ _TIMED = ("embed_gather", "feed_tokens", "add_rmsnorm", "residual_add", "swiglu"
           "router_topk", "router", "moe_plan", "moe_gate_up", "moe_down", "moe_combine", "branch_norm_add", "stream_add",
           "qk_joint_norm_rope_store", "gla_scan", "gla_norm_gate", "linear_scan", "rows_dot_f32", "mlstm_gate_scan", "mlstm_norm_gate",
           "ssm_conv", "ssm_gate_norm", "scale_rows", "weighted_sum", "rope_table", "qkv_prepare", "gate_rows", "causal_conv", "delta_scan",
+          "channel_decay", "rotate_qkv",
           "softcap_rows", "rglru_scan", "rglru_step", "rmsnorm_rows", "library_bmm_float32")
 _plain_functions: dict[str, object] = {}
 _kernel_events: list[tuple[str, "torch.cuda.Event", "torch.cuda.Event"]] = []

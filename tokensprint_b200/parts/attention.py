@@ -57,9 +57,13 @@ class AttentionMixer(Mixer):
     `distance` = (name r1, name r2) of two [num_heads] tensors: the scaled score of key j for the query
     at position i loses r1_h * ln(1 + r2_h * (i - j)), a penalty per head that grows with the logarithm
     of the distance (positions enter such a layer through it, and through the temperature, alone).
+    `gate_per` = "head": the gate matrix has one row per head, and a whole head is multiplied by one sigmoid.
+    `shares_values` = key: this layer's values (before any blending) are kept until the end of the step under
+    that key; `value_mix` = (key, name of a single number m): the values that are stored and attended to are
+    (1 - m) v + m times those kept under the key for the same tokens by an earlier layer.
     A position encoding whose cosines and sines carry a magnitude is applied from its table.
     With any of the options from `sinks` on, one product gives [q | k | v | gate], `qkv_prepare`
-    adds biases, rotates, norms and stores (keys and values padded with zeros to one common width
+    adds biases, norms (the weighted norm per head before the rotation, the unit norm behind it), rotates and stores (keys and values padded with zeros to one common width
     that the attention kernels take), and the gate is a kernel behind attention.
     """
 
@@ -99,6 +103,9 @@ class AttentionMixer(Mixer):
         gate: Optional[str] = None,
         q_temperature: Optional[Sequence[float]] = None,
         distance: Optional[Sequence[str]] = None,
+        gate_per: str = "entry",
+        shares_values: Optional[str] = None,
+        value_mix: Optional[Sequence[str]] = None,
     ) -> None:
         if qk_norm is True:
             qk_norm = "head"
@@ -138,6 +145,14 @@ class AttentionMixer(Mixer):
         self.names = {"q": q, "k": k, "v": v, "o": o, "q_norm": q_norm, "k_norm": k_norm, "sinks": sinks, "q_bias": q_bias,
                       "k_bias": k_bias, "v_bias": v_bias, "gate": gate,
                       "r1": None if distance is None else distance[0], "r2": None if distance is None else distance[1]}
+        if gate_per not in ("entry", "head"):
+            raise ValueError(f"attention: gate_per must be 'entry' or 'head', got {gate_per!r}")
+        if value_mix is not None and len(value_mix) != 2:
+            raise ValueError("attention: value_mix is (key, tensor name)")
+        self.gate_per_head = gate_per == "head"
+        self.shares_values = shares_values
+        self.value_mix = None if value_mix is None else (value_mix[0], value_mix[1])
+        self.value_share = 0.0
         self.q_temperature = None if q_temperature is None else (float(q_temperature[0]), int(q_temperature[1]))
         self.distance: Optional[tuple[torch.Tensor, torch.Tensor]] = None
         self.position = build_part("position_encoding", position, ctx) if position is not None else None
@@ -146,14 +161,14 @@ class AttentionMixer(Mixer):
         magnitude = getattr(self.position, "magnitude", 1.0) if self.position is not None else 1.0
         # the path through qkv_prepare (see the class's text)
         self.general = bool(unit_after or sinks or softcap or q_bias or k_bias or v_bias or gate or self.value_dim != self.head_dim
-                            or magnitude != 1.0 or q_temperature is not None or distance is not None)
+                            or magnitude != 1.0 or q_temperature is not None or distance is not None or shares_values or value_mix)
         # the width the attention kernels run at: the wider of keys and values, and in bfloat16 the next
         # multiple of 16 (what the tensor-core kernels take): entries beyond a head's own are zeros
         self.kernel_dim = self.head_dim
         if self.general:
-            if self.joint_norm or self.qk_norm or self.values_are_keys:
+            if self.joint_norm or self.values_are_keys or (self.qk_norm and unit_after):
                 raise ValueError("attention: biases, a unit norm after the rotation, a gate, learned sinks, a score cap and values of "
-                                 "another width come without the weighted q/k norms and with a value projection")
+                                 "another width come without the norm over the whole projection and with a value projection")
             if self.position is not None and not hasattr(self.position, "rotary_table"):
                 raise ValueError("attention: these options take a rotation that offers its table of cosines and sines (or none)")
             self.kernel_dim = max(self.head_dim, self.value_dim)
@@ -197,7 +212,9 @@ class AttentionMixer(Mixer):
         if not self.values_are_keys:
             specs.insert(2, TensorSpec(self.names["v"], (nkv * e, H)))
         if n["gate"] is not None:
-            specs.append(TensorSpec(n["gate"], (nq * e, H)))
+            specs.append(TensorSpec(n["gate"], (nq if self.gate_per_head else nq * e, H)))
+        if self.value_mix is not None:
+            specs.append(TensorSpec(self.value_mix[1], (), "vector"))
         if n["sinks"] is not None:
             specs.append(TensorSpec(n["sinks"], (nq,), "vector"))
         if n["r1"] is not None:
@@ -225,6 +242,8 @@ class AttentionMixer(Mixer):
         for key in ("q", "k", "v"):
             if n[key + "_bias"] is not None:
                 self.biases[key] = tensors[n[key + "_bias"]]
+        if self.value_mix is not None:
+            self.value_share = float(tensors[self.value_mix[1]])
         self.o_weight = tensors[n["o"]]
         if self.qk_norm:
             self.q_norm_weight = tensors[n["q_norm"]]
@@ -302,8 +321,8 @@ class AttentionMixer(Mixer):
         return linear(out, self.o_weight, next_weight=step.weight_after)
 
     def _forward_general(self, x, step: StepContext, cache: LayerCache, tables):
-        """One product for [q | k | v | gate]; biases, rotation from the table, the unit norm and the
-        stores in one kernel (keys and values padded to the kernels' width); attention; the gate
+        """One product for [q | k | v | gate]; biases, weighted norms, rotation from the table, the unit norm, the
+        blend of the values and the stores in one kernel (keys and values padded to the kernels' width); attention; the gate
         (and the cut back to the values' own width); the output product."""
         T = x.shape[0]
         nq, nkv, d, e, D = self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim, self.kernel_dim
@@ -312,16 +331,21 @@ class AttentionMixer(Mixer):
         q = torch.empty((T, nq * D), device=x.device, dtype=x.dtype)
         k_off, v_off, g_off = nq * d, nq * d + nkv * d, nq * d + nkv * d + nkv * e
         writes = cache.writes
+        if self.shares_values is not None:
+            step.shared["values", self.shares_values] = proj[:, v_off:g_off]
+        first = step.shared["values", self.value_mix[0]] if self.value_mix is not None else None
         ops.qkv_prepare(proj, 0, k_off, v_off, self.biases["q"], self.biases["k"], self.biases["v"], table, self.unit_after_rotation,
                         self.qk_norm_eps, q, cache.k_pages if writes else None, cache.v_pages if writes else None,
                         tables.slot_mapping if writes else None, nq, nkv, d, e, D, positions=step.positions,
-                        query_temperature=self.q_temperature)
+                        query_temperature=self.q_temperature, q_norm=self.q_norm_weight, k_norm=self.k_norm_weight,
+                        first_values=first, value_share=self.value_share)
         out = torch.empty((T, nq * D), device=x.device, dtype=x.dtype)
         self._attend(q, out, step, cache, tables)
         gated = self.names["gate"] is not None
         if gated or D != e:
             y = torch.empty((T, nq * e), device=x.device, dtype=x.dtype)
-            ops.gate_rows(out, proj[:, g_off:g_off + nq * e] if gated else None, y, nq, e, D)
+            ops.gate_rows(out, proj[:, g_off:g_off + (nq if self.gate_per_head else nq * e)] if gated else None, y, nq, e, D,
+                          per_head=self.gate_per_head)
             out = y
         return linear(out, self.o_weight, next_weight=step.weight_after)
 

@@ -3,7 +3,7 @@ with capped operands, a layer of routed experts of that form, and a per-layer to
 
 from __future__ import annotations
 
-from typing import Mapping, Optional
+from typing import Mapping, Optional, Sequence
 
 import torch
 
@@ -91,6 +91,9 @@ class RoutedExperts(FeedForward):
                  "softmax_all": scores s = softmax(z) over all experts; the `top` largest of
                  s + c are chosen (`correction` names c, a number per expert that steers the choice
                  only) and the weights are the chosen s themselves (divided by their sum with `renormalize`)
+        `groups` = (count, keep): the experts form `count` equal groups of neighbours; only those of the `keep` groups
+                    whose best member is largest may be chosen
+        `weight_scale`: a constant on every weight, after the division by their sum
         f = sum over chosen e of expert_e(w_e x)   (`weight_on` "input"; "output": w_e expert_e(x))
             + shared(x) if a shared expert is named (any feed-forward spec)
         expert(x) = W_down act(W_gate x, W_up x), `activation` "capped_glu" (with `limit`, `alpha`)
@@ -111,7 +114,8 @@ class RoutedExperts(FeedForward):
     def __init__(self, ctx: BuildContext, *, hidden_size: int, num_experts: int, top: int, intermediate_size: int,
                  router: str, expert_prefix: str, limit: float = 0.0, alpha: float = 1.702, renormalize: bool = False,
                  weight_on: str = "input", shared: Optional[PartSpec] = None, router_bias: Optional[str] = None,
-                 score: str = "sigmoid", activation: str = "capped_glu", correction: Optional[str] = None, identity: int = 0) -> None:
+                 score: str = "sigmoid", activation: str = "capped_glu", correction: Optional[str] = None, identity: int = 0,
+                 groups: Optional[Sequence[int]] = None, weight_scale: float = 1.0) -> None:
         self.hidden_size, self.num_experts, self.top = int(hidden_size), int(num_experts), int(top)
         self.intermediate_size, self.limit, self.alpha = int(intermediate_size), float(limit), float(alpha)
         self.renormalize = bool(renormalize)
@@ -131,6 +135,13 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"routed experts: top {top} of {num_experts} + {identity} router outputs")
         if correction is not None and score != "softmax_all":
             raise ValueError("routed experts: a correction of the choice comes with score = 'softmax_all'")
+        self.weight_scale = float(weight_scale)
+        self.groups = None if groups is None else (int(groups[0]), int(groups[1]))
+        if self.groups is not None:
+            count, keep = self.groups
+            outputs = self.num_experts + self.identity
+            if count < 1 or outputs % count or not 1 <= keep <= count or self.top > keep * (outputs // count):
+                raise ValueError(f"routed experts: {keep} of {count} groups of {outputs} experts cannot give {top} choices")
         self.gated = activation != "gelu"
         self.correction_name = correction
         self.correction: Optional[torch.Tensor] = None
@@ -182,7 +193,8 @@ class RoutedExperts(FeedForward):
         rows = residual if residual is not None else x  # float32 rows where the block has them, else their rounding
         chosen = torch.empty((T, top), device=dev, dtype=torch.int32)
         weights = torch.empty((T, top), device=dev, dtype=torch.float32)
-        ops.router(rows, self.router, top, self.renormalize, chosen, weights, bias=self.router_bias, score=self.score, correction=self.correction)
+        ops.router(rows, self.router, top, self.renormalize, chosen, weights, bias=self.router_bias, score=self.score, correction=self.correction,
+                   groups=self.groups, scale=self.weight_scale)
         # both products take the same plan: the tensor cores only if both inner widths suit them
         tensor_cores = ops.moe_on_tensor_cores(x.dtype, self.hidden_size, self.intermediate_size)
         plan = ops.moe_plan(chosen, self.num_experts, ops.moe_row_tile(tensor_cores, T * top, self.num_experts))

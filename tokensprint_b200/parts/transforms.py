@@ -47,6 +47,30 @@ class PairHashEmbedding(Transform):
         return x
 
 
+@register_part("transform", "rmsnorm")
+class RowNorm(Transform):
+    """x <- x * rsqrt(mean(x^2) + eps) * weight row by row in float32: a norm on the embedding rows before the
+    first block reads them as the residual stream."""
+
+    graph_safe = True
+    reads_through_ops = True
+
+    def __init__(self, ctx: BuildContext, *, dim: int, eps: float, weight: str) -> None:
+        self.dim, self.eps, self.name = int(dim), float(eps), weight
+        self.weight: Optional[torch.Tensor] = None
+
+    def tensor_specs(self) -> list[TensorSpec]:
+        return [TensorSpec(self.name, (self.dim,), "vector")]
+
+    def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        self.weight = tensors[self.name]
+
+    def forward(self, x: torch.Tensor, step: Optional[StepContext]) -> torch.Tensor:
+        out = torch.empty_like(x)
+        ops.add_rmsnorm(x, None, self.weight, out, self.eps)
+        return out
+
+
 @register_part("transform", "pass_entry")
 class PassEntry(Transform):
     """What a model adds to the residual stream where a stretch of layers begins (a model that runs
