@@ -408,7 +408,7 @@ def run_probe(args) -> int:
         from tokensprint_b200.config.registry import get_model_config
 
         cfg = get_model_config({"dazilix": "dazilix-w2048", "pekunex": "pekunex-w2048", "vasosun": "vasosun-w2048",
-                                "mugulorn": "mugulorn-w2048"}.get(args.designs, "fegetar-w2048"))
+                                "mugulorn": "mugulorn-w2048", "vepevik": "vepevik-w2048"}.get(args.designs, "fegetar-w2048"))
     else:
         d = get_preset_dict(MODEL_NAME)
         d["num_hidden_layers"] = args.layers or 4
@@ -743,10 +743,10 @@ def main() -> int:
                         "(the events cost host time: take the throughput from a run without this option)")
     p.add_argument("--workload", choices=sorted(WORKLOADS), default=None,
                    help="a serving loop through generate() instead of the decode benchmark (one JSON line)")
-    p.add_argument("--designs", nargs="?", const="fegetar", default=None, choices=["fegetar", "dazilix", "pekunex", "vasosun", "mugulorn"],
+    p.add_argument("--designs", nargs="?", const="fegetar", default=None, choices=["fegetar", "dazilix", "pekunex", "vasosun", "mugulorn", "vepevik"],
                    help="another design beside Qwen3 dense at equal size (a few layers of realistic widths, random weights): prompt and "
                         "decode throughput and the design's kernels against their rooflines (one JSON line); "
-                        "without a name: Fegetar; pekunex and vasosun run beside Dazilix, mugulorn beside Vasosun, the closest designs")
+                        "without a name: Fegetar; pekunex and vasosun run beside Dazilix, mugulorn beside Vasosun, vepevik beside both, the closest designs")
     p.add_argument("--probe", choices=["decode", "prefill"], default=None,
                    help="run a few steps inside cudaProfilerStart/Stop for ncu and exit (see profiles/); with --designs: of Fegetar's named model")
     args = p.parse_args()

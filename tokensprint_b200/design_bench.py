@@ -31,6 +31,13 @@ feed-forward, gelu feed-forwards) beside Vasosun, the closest design the engine 
 attention, a recurrence), put together from the same kinds of layers at equal sizes: latent attention,
 its reader, two delta layers, dense feed-forwards where Mugulorn has them; with the distance of both
 designs' kernels from their rooflines.
+
+`python bench.py --designs vepevik` runs Vepevik (attention inside chunks with normed q and k, blended values
+and a gate per head; retention; the delta rule with a decay per key channel; a capped dense feed-forward and
+routed experts chosen inside groups) beside the two designs it is closest to, put together from the same kinds of
+layers at equal sizes: Dazilix (attention inside blocks, gated linear attention, routed experts of the same sizes)
+and Vasosun (the delta rule with one decay per head), with the distance of all three designs' kernels
+from their rooflines.
 """
 
 from __future__ import annotations
@@ -200,6 +207,108 @@ def vasosun_beside_mugulorn(s: dict) -> dict:
             "embedding": {"bigram": {"buckets": 65521, "mul_prev": 1000003, "mul_cur": 31}}, "logit_softcap": 30.0,
             "layers": [{"type": "latent_attention", "mixer": lat, "mlp": mlp},
                        {"type": "latent_attention", "mixer": dict(lat, kv_from=0), "mlp": mlp}, delta, delta]}
+
+
+# Vepevik at the same widths: two attention layers (heads of 128, a chunk that holds the prompt), a retention of Dazilix's
+# recurrent sizes, a delta layer of Vasosun's; the first feed-forward dense with the weight per token of the chosen experts,
+# the others routed, with four groups of experts of which two are kept.
+VEPEVIK_SIZES = {
+    "w2048": dict(width=2048, heads=16, layers=4, experts=16, top=2, expert_ff=1024, gla_dim=64, gla_vdim=128, delta_dim=64, delta_vdim=128,
+                  block=4096, window=4096, taps=4, rank=64),
+    "w4096": dict(width=4096, heads=32, layers=4, experts=32, top=4, expert_ff=1536, gla_dim=64, gla_vdim=128, delta_dim=64, delta_vdim=128,
+                  block=4096, window=4096, taps=4, rank=64),
+}
+
+
+def vepevik_config(s: dict) -> dict:
+    H = s["heads"]
+    att = {"heads": H, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "rot": {"base": 1000000.0, "dims": 64},
+           "mask": {"size": s["block"]}, "v_mix": True}
+    ret = {"heads": H, "dim": s["gla_dim"], "vdim": s["gla_vdim"], "decay": [1.0 - 2.0 ** (-5 - 7 * h / H) for h in range(H)],
+           "rot": {"base": 10000.0, "dims": s["gla_dim"]}}
+    delta = {"heads": H, "kv_heads": H, "dim": s["delta_dim"], "vdim": s["delta_vdim"], "conv": s["taps"], "decay_rank": s["rank"], "gate_rank": s["rank"]}
+    dense = {"kind": "dense", "ff": s["top"] * s["expert_ff"], "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": s["expert_ff"]},
+           "router": {"experts": s["experts"], "top": s["top"], "scale": 2.5, "groups": {"count": 4, "keep": 2}}}
+    return {"architecture": "Vepevik", "vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-6},
+            "layers": [{"type": "attention", "mixer": att, "mlp": dense}, {"type": "retention", "mixer": ret, "mlp": moe},
+                       {"type": "channel_delta", "mixer": delta, "mlp": moe}, {"type": "attention", "mixer": att, "mlp": moe}]}
+
+
+def dazilix_beside_vepevik(s: dict) -> dict:
+    d = dazilix_config(s)
+    att, gla = d["layers"][0], d["layers"][DAZILIX_RECURRENT_LAYERS[0]]
+    return dict(d, layers=[att, gla, gla, att])
+
+
+def vasosun_beside_vepevik(s: dict) -> dict:
+    att = {"heads": s["heads"], "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": s["window"]}}
+    delta = {"heads": s["heads"], "kv_heads": s["heads"], "dim": s["delta_dim"], "vdim": s["delta_vdim"], "conv": s["taps"]}
+    moe = {"kind": "moe", "expert": {"ff": s["expert_ff"]}, "router": {"experts": s["experts"], "identity": 0, "top": s["top"]}}
+    layers = [{"type": t, "mixer": m, "mlp": moe} for t, m in (("attention", att), ("delta", delta), ("delta", delta), ("attention", att))]
+    return {"architecture": "Vasosun", "vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-6}, "canon": {"taps": s["taps"]},
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 1000003, "mul_cur": 31}}, "logit_softcap": 30.0, "layers": layers}
+
+
+def _vepevik_rooflines(design: str, s: dict, m: dict, peaks: dict) -> dict[str, Any]:
+    """The three designs' kernels against their rooflines, from the per-class timers, all layers of a step summed.
+    Attention: 4 * 128 operations per (query, key, head) against the bf16 peak; a decode step reads every cached row
+    once.  Recurrences: a linear one costs 6 float32 operations per state entry and token, the delta rule 8, against
+    the FFMA rate of the SMs at their top clock; a decode step reads and writes every request's states once, against the
+    measured copy bandwidth.  The other kernels move their inputs and outputs once, against the same."""
+    out: dict[str, Any] = {}
+    H, W, T = s["heads"], s["width"], PREFILL_TOKENS
+    hbm, bf16 = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    ffma_peak = 148 * 128 * 2 * peaks.get("sm_max_mhz", 1965.0) * 1e6
+    gd, gv, dd, dv = s["gla_dim"], s["gla_vdim"], s["delta_dim"], s["delta_vdim"]
+    chans = H * (2 * dd + dv)
+    attention_names = ("attention_prefill_tcgen05", "attention_paged_mma", "attention_paged_simple")
+    if design == "vepevik":
+        scans = {"linear_scan": (1, H * gd * gv, 6.0), "delta_scan": (1, H * dd * dv, 8.0)}  # layers, state entries, operations
+        small = {  # bytes per token
+            "add_rmsnorm": (2 * s["layers"]) * W * 12 + W * 8, "qkv_prepare": 2 * 2 * (H + 16) * 128 * 2 + 8 * 128 * 2, "gate_rows": 2 * 2 * H * 128 * 2,
+            "rotate_qkv": H * (2 * gd + gv) * (2 + 4), "causal_conv": chans * (2 + 4), "channel_decay": H * dd * 8,
+            "gla_norm_gate": H * gv * (4 + 2 + 2) + H * dv * (4 + 4 + 2), "capped_glu": 3 * s["top"] * s["expert_ff"] * 2,
+            "moe_combine": 3 * (s["top"] + 1) * W * 2, "router": 3 * W * 2,
+        }
+    elif design == "dazilix":
+        scans = {"gla_scan": (2, H * gd * gv, 6.0)}
+        small = {
+            "branch_norm_add": 2 * s["layers"] * W * 12, "qk_joint_norm_rope_store": 2 * (2 * H + 3 * 8) * 128 * 2, "gla_norm_gate": 2 * H * gv * (4 + 2 + 2),
+            "moe_combine": 4 * (s["top"] + 1) * W * 2, "router": 4 * W * 2,
+        }
+    else:
+        scans = {"delta_scan": (2, H * dd * dv, 8.0)}
+        small = {
+            "branch_norm_add": 2 * s["layers"] * W * 12, "qkv_prepare": 2 * 2 * (H + 16) * 128 * 2,
+            "causal_conv": 2 * s["layers"] * W * (2 + 2) + 2 * chans * (2 + 4), "gla_norm_gate": 2 * H * dv * (4 + 2 + 2),
+            "moe_combine": 4 * (s["top"] + 1) * W * 2, "router": 4 * W * 2,
+        }
+    steps = [("prefill", m["prefill_kernels"], T)] + [(f"decode_b{b}", m[f"decode_b{b}_kernels"], b) for b in DECODE_BATCHES]
+    for phase, kernels, tokens in steps:
+        prompt = phase == "prefill"
+        ms = sum(v["ms"] for k, v in kernels.items() if k in attention_names)
+        if ms > 0:
+            out[f"{phase}_attention_ms"] = round(ms, 4)
+            if prompt:
+                out["prefill_attention_of_bf16_peak"] = round(2 * 4 * H * 128 * T * (T + 1) / 2 / (ms * 1e-3) / bf16, 3)
+            else:
+                out[f"{phase}_attention_of_hbm_peak"] = round(2 * tokens * DECODE_CONTEXT * 2 * 8 * 128 * 2 / (ms * 1e-3) / hbm, 3)
+        for name, (layers, entries, per_entry) in scans.items():
+            ms = kernels.get(name, {}).get("ms", 0.0)
+            if ms > 0:
+                out[f"{phase}_{name}_ms"] = round(ms, 4)
+                if prompt:
+                    out[f"prefill_{name}_of_ffma_peak"] = round(layers * per_entry * T * entries / (ms * 1e-3) / ffma_peak, 3)
+                else:
+                    out[f"{phase}_{name}_of_hbm_peak"] = round(layers * tokens * entries * 8 / (ms * 1e-3) / hbm, 3)
+        for name, per_token in small.items():
+            ms = kernels.get(name, {}).get("ms", 0.0)
+            if ms > 0:
+                out[f"{phase}_{name}_ms"] = round(ms, 4)
+                if prompt:
+                    out[f"prefill_{name}_of_hbm_peak"] = round(tokens * per_token / (ms * 1e-3) / hbm, 3)
+    return out
 
 
 def _mugulorn_rooflines(design: str, s: dict, m: dict, peaks: dict) -> dict[str, Any]:
@@ -522,10 +631,13 @@ def run(steps: int, warmup: int, peaks: dict, which: str = "fegetar") -> dict[st
 
     result: dict[str, Any] = {"metric": "design_comparison", "dtype": "bf16", "data": "synthetic, random weights",
                               "prefill_tokens": PREFILL_TOKENS, "decode_context": DECODE_CONTEXT, "sizes": {}}
-    sizes = {"dazilix": DAZILIX_SIZES, "pekunex": PEKUNEX_SIZES, "vasosun": VASOSUN_SIZES, "mugulorn": MUGULORN_SIZES}.get(which, SIZES)
+    sizes = {"dazilix": DAZILIX_SIZES, "pekunex": PEKUNEX_SIZES, "vasosun": VASOSUN_SIZES, "mugulorn": MUGULORN_SIZES,
+             "vepevik": VEPEVIK_SIZES}.get(which, SIZES)
     for name, s in sizes.items():
         row: dict[str, Any] = {"size": s}
-        if which == "mugulorn":
+        if which == "vepevik":
+            pair = (("vepevik", vepevik_config(s)), ("dazilix", dazilix_beside_vepevik(s)), ("vasosun", vasosun_beside_vepevik(s)))
+        elif which == "mugulorn":
             pair = (("mugulorn", mugulorn_config(s)), ("vasosun", vasosun_beside_mugulorn(s)))
         elif which == "vasosun":
             pair = (("vasosun", vasosun_config(s)), ("dazilix", dazilix_beside_vasosun(s)))
@@ -541,9 +653,11 @@ def run(steps: int, warmup: int, peaks: dict, which: str = "fegetar") -> dict[st
             m = _measure(model, steps, warmup)
             m["weight_bytes"] = model.weight_bytes()
             sd = DAZILIX_SIZES[name] if (which in ("pekunex", "vasosun") and design == "dazilix") else s
-            if which != "mugulorn":
+            if which not in ("mugulorn", "vepevik"):
                 m.update(_attention_rooflines(design, sd, m, peaks))
-            if which == "mugulorn":
+            if which == "vepevik":
+                m.update(_vepevik_rooflines(design, s, m, peaks))
+            elif which == "mugulorn":
                 m.update(_mugulorn_rooflines(design, s, m, peaks))
             elif which == "vasosun":
                 m.update(_vasosun_rooflines(s, m, peaks) if design == "vasosun" else _dazilix_rooflines(sd, m, peaks))
