@@ -92,7 +92,8 @@ def _delta_run(x, gates, a_log, dt_bias, state, slots, lengths, H, G, d, e):
     out = torch.empty((x.shape[0], H * e), device="cuda")
     rows = _dev(gates)
     ops.delta_scan(_dev(x), 0, G * d, 2 * G * d, rows[:, :H], rows[:, H:], _dev(a_log), _dev(dt_bias), state, _i32(slots), cu, out, len(lengths),
-                   H, G, d, e, d ** -0.5, 1e-6)
+                   H, G, d, e, d ** -0.5, 1e-6,
+                   max_seqlen=max(lengths))
     return out.cpu()
 
 

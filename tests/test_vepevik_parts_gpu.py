@@ -59,7 +59,8 @@ def _delta_run(data, state, slots, lengths, H, G, d, e, ahead, beta_dtype=torch.
         ops.channel_decay(rows, a_log, dt_bias, H, d)
         a_log = dt_bias = None
     out = torch.empty((x.shape[0], H * e), device="cuda")
-    ops.delta_scan(_dev(x), 0, G * d, 2 * G * d, betas, rows, a_log, dt_bias, state, _i32(slots), cu, out, len(lengths), H, G, d, e, d ** -0.5, 1e-6)
+    ops.delta_scan(_dev(x), 0, G * d, 2 * G * d, betas, rows, a_log, dt_bias, state, _i32(slots), cu, out, len(lengths), H, G, d, e, d ** -0.5, 1e-6,
+                   max_seqlen=max(lengths))
     return out.cpu()
 
 

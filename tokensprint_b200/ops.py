@@ -1168,9 +1168,6 @@ def rglru_step(u: torch.Tensor, gates: torch.Tensor, bias_r: torch.Tensor, bias_
 
 
 DELTA_MAX_KEY_DIM = 1024
-# TS_DELTA_LANES (for measurements): lanes that share a value column of the delta rule's state (a power of two up to 32);
-# unset or 0: the kernel's own choice by the key width
-DELTA_LANES = int(_os.environ.get("TS_DELTA_LANES", "0"))
 
 
 def channel_decay(z: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, num_heads: int, key_dim: int) -> None:
@@ -1189,7 +1186,8 @@ def channel_decay(z: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, n
 
 def delta_scan(x: torch.Tensor, q_off: int, k_off: int, v_off: int, beta: torch.Tensor, decay: torch.Tensor, a_log: Optional[torch.Tensor],
                dt_bias: Optional[torch.Tensor], state: torch.Tensor, state_slots: torch.Tensor, cu_seqlens: torch.Tensor, out: torch.Tensor,
-               num_seqs: int, num_heads: int, num_qk_heads: int, key_dim: int, value_dim: int, q_scale: float, unit_eps: float) -> None:
+               num_seqs: int, num_heads: int, num_qk_heads: int, key_dim: int, value_dim: int, q_scale: float, unit_eps: float,
+               max_seqlen: Optional[int] = None) -> None:
     """The gated delta rule over the tokens of every sequence, in order (csrc/delta_rule.cu).  x [T, n]
     float32 holds q (columns q_off.., num_qk_heads * key_dim), k (k_off..) and v (v_off.., num_heads *
     value_dim); q and k are brought to unit length per head here and q is multiplied by q_scale.
@@ -1198,7 +1196,8 @@ def delta_scan(x: torch.Tensor, q_off: int, k_off: int, v_off: int, beta: torch.
     per column of decay) the raw rows, of which exp(-exp(a_log) * softplus(raw + dt_bias)) is taken here;
     with None for both the decays themselves.  beta and decay may be column ranges of wider matrices.
     state [slots, >= heads * value_dim * key_dim] float32 (a view with a row stride is fine), one head after the
-    other, value column by value column; out [T, heads * value_dim] float32."""
+    other, value column by value column; out [T, heads * value_dim] float32.  `max_seqlen`: the most tokens a
+    sequence brings; 1 runs the tokens singly, otherwise they go through in blocks."""
     flush_gemm_chain()
     H, G, d, e = int(num_heads), int(num_qk_heads), int(key_dim), int(value_dim)
     T = x.shape[0]
@@ -1226,7 +1225,7 @@ def delta_scan(x: torch.Tensor, q_off: int, k_off: int, v_off: int, beta: torch.
     _check("delta_scan", _fn("ts_delta_scan")(
         x.data_ptr(), x.stride(0), int(q_off), int(k_off), int(v_off), beta.data_ptr(), _act_code("beta", beta), beta.stride(0), decay.data_ptr(),
         decay.stride(0), 1 if per_channel else 0, 0 if a_log is None else 1, _ptr(a_log), _ptr(dt_bias), state.data_ptr(), state.stride(0),
-        state_slots.data_ptr(), cu_seqlens.data_ptr(), out.data_ptr(), int(num_seqs), H, G, d, e, float(q_scale), float(unit_eps), DELTA_LANES,
+        state_slots.data_ptr(), cu_seqlens.data_ptr(), out.data_ptr(), int(num_seqs), H, G, d, e, float(q_scale), float(unit_eps), 1 if max_seqlen == 1 else 0,
         _stream()))
 
 

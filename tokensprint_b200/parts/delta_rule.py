@@ -160,7 +160,7 @@ class GatedDeltaRule(Mixer):
             a_log = dt_bias = None
         o = torch.empty((T, self.v_width), device=x.device, dtype=torch.float32)
         ops.delta_scan(conv, 0, self.qk_width, 2 * self.qk_width, beta, decay, a_log, dt_bias, state, step.state_slots, step.cu_seqlens_q, o,
-                       step.num_seqs, H, G, d, e, self.q_scale, self.unit_eps)
+                       step.num_seqs, H, G, d, e, self.q_scale, self.unit_eps, max_seqlen=step.max_seqlen_q)
         y = torch.empty((T, self.v_width), device=x.device, dtype=x.dtype)
         ops.gla_norm_gate(o, gate, self.norm_weight, y, H, e, self.norm_eps, activation=self.gate_activation)
         return linear(y, self.o_weight, next_weight=step.weight_after)
