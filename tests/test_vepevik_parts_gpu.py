@@ -120,14 +120,14 @@ def test_a_channel_that_forgets_at_once_and_one_that_never_does():
             assert _rel(got, want) < 3e-5, (ahead, n)
 
 
-RETENTION_SHAPES = [([0.9], 7, 5, 6), ([0.5, 1.0, 0.97], 20, 11, 8), ([0.99, 0.75], 64, 64, 64), ([0.998] * 4, 130, 36, 0)]
+RETENTION_SHAPES = [([0.9], 7, 5, 6), ([0.5, 1.0, 0.97], 20, 11, 8), ([0.99, 0.75], 64, 64, 64), ([0.998] * 4, 130, 36, 0), ([0.9, 0.99], 15, 20, 2),
+                    ([0.96875], 60, 33, 34), ([0.9], 128, 40, 128), ([0.5, 0.99], 100, 17, 70), ([0.99], 300, 24, 260), ([0.9, 1.0], 2, 70, 2)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("decay, d, e, rot", RETENTION_SHAPES)
-def test_constant_decay_scan_in_portions_token_by_token_and_in_segments(decay, d, e, rot, dtype):
-    """Rotated float32 rows (portions) and rows rotated as they are read (single tokens) against the plain recurrence;
-    1,100 tokens run in segments side by side."""
+def test_retention_scan_whole_in_portions_and_token_by_token(decay, d, e, rot, dtype):
+    """Rows that are rotated as they are read (all of a head, its first entries, none) against the plain recurrence."""
     from tokensprint_b200 import ops
 
     H, T = len(decay), 1100
@@ -144,17 +144,50 @@ def test_constant_decay_scan_in_portions_token_by_token_and_in_segments(decay, d
         while at < T and not (sizes == (1,) and at >= 120):
             n = min(sizes[i % len(sizes)], T - at)
             table = ops.rope_table(_i32(pos[at:at + n]), _dev(inv), 1.0, n) if rot else None
-            part = rows[at:at + n]
-            if n > 1:
-                part, table = ops.rotate_qkv(part, 0, H * d, 2 * H * d, table, H, d, e), None
             o = torch.empty((n, H * e), device="cuda")
-            ops.linear_scan(part[:, :H * d], part[:, H * d:2 * H * d], part[:, 2 * H * d:H * (2 * d + e)], constants, None, d ** -0.5, state,
-                            _i32([1]), _i32([0, n]), o, 1, H, H, d, e, max_seqlen=n, rotation=table)
+            ops.retention_scan(rows[at:at + n], 0, H * d, 2 * H * d, table, constants, d ** -0.5, state, _i32([1]), _i32([0, n]), o, 1, H, H, d, e,
+                               max_seqlen=n)
             out.append(o.cpu())
             at, i = at + n, i + 1
         got = torch.cat(out)
         assert _rel(got, want[:got.shape[0]]) < 5e-5, sizes
         assert float(state[[0, 2]].abs().max()) == 0.0 and float(state[1, H * d * e:].abs().max()) == 0.0
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H, G, d, e, rot", [(6, 2, 12, 10, 4), (4, 4, 64, 64, 64), (4, 1, 40, 70, 0)])
+def test_retention_scan_many_sequences_side_by_side_against_each_alone(H, G, d, e, rot, dtype):
+    """Thirty sequences of unequal length (one of them empty) in one launch, q and k heads shared by groups of value heads,
+    slots in any order; then one more token of each."""
+    from tokensprint_b200 import ops
+
+    lengths = [(7 * i) % 23 + 1 for i in range(30)]
+    lengths[5] = 0
+    decay = [1.0 - 0.5 ** (h + 1) for h in range(H)]
+    xs = [_rand((n + 1, 2 * G * d + H * e), 200 + i).to(dtype) for i, n in enumerate(lengths)]
+    want = []
+    for x in xs:
+        p, pos = x.double(), list(range(x.shape[0]))
+        q, k = (plain.rotate_half(p[:, a:a + G * d].view(-1, G, d), pos, 50.0, rot) for a in (0, G * d))
+        v = p[:, 2 * G * d:].view(-1, H, e)
+        want.append(torch.cat([plain.retention_recurrence(q[:, a // (H // G)] * d ** -0.5, k[:, a // (H // G)], v[:, a], decay[a]) for a in range(H)], -1))
+    state = torch.zeros((30, H * d * e), device="cuda")
+    slots = [(7 * i) % 30 for i in range(30)]
+    state[slots[5]] = 3.0
+    inv = torch.as_tensor(50.0, dtype=torch.float64) ** (-2.0 * torch.arange(rot // 2, dtype=torch.float64) / max(rot, 1))
+    for first in (True, False):
+        parts = [(0, n) if first else (n, n + 1) for n in lengths]
+        if not first:
+            parts[5] = (0, 0)
+        rows = torch.cat([x[a:b] for x, (a, b) in zip(xs, parts)])
+        pos = [t for a, b in parts for t in range(a, b)]
+        cu, _ = _batch([b - a for a, b in parts])
+        out = torch.empty((rows.shape[0], H * e), device="cuda")
+        table = ops.rope_table(_i32(pos), _dev(inv), 1.0, len(pos)) if rot else None
+        ops.retention_scan(_dev(rows), 0, G * d, 2 * G * d, table, torch.tensor(decay, device="cuda"), d ** -0.5, state, _i32(slots), cu, out, 30, H, G,
+                           d, e, max_seqlen=max(b - a for a, b in parts))
+        assert _rel(out.cpu(), torch.cat([w[a:b] for w, (a, b) in zip(want, parts)])) < 3e-5, first
+    assert float((state[slots[5]] - 3.0).abs().max()) == 0.0  # the empty lane's slot
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -194,7 +227,7 @@ def test_norms_rotation_and_blended_values_between_projection_and_cache(dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("T, H, e, D", [(7, 5, 12, 16), (9, 2, 64, 64), (3, 3, 9, 9)])
+@pytest.mark.parametrize("T, H, e, D", [(7, 5, 12, 16), (9, 2, 64, 64), (3, 3, 9, 9), (70, 3, 40, 40)])
 def test_one_gate_per_head(T, H, e, D, dtype):
     from tokensprint_b200 import ops
 
@@ -452,7 +485,7 @@ def test_values_blended_with_the_first_layers(tag, layer, dtype):
 @pytest.mark.parametrize("layer", [1, 2])
 def test_a_far_key_through_the_recurrences(layer, dtype):
     """Only the first tokens carry input, the hundreds behind them (almost) none but their queries: what they read out is
-    what the state still holds, in one piece, in segments, over cuts and one by one."""
+    what the state still holds, in one piece, over cuts and one by one."""
     cfg = VEP_LONG
     parts, W = _layer_parts(cfg, layer, dtype, 26, 1.0, RANKS["long"])
     f = _plain_mixer(cfg, layer, W)

@@ -159,7 +159,7 @@ def test_long_decoding_with_graphs_and_without(models, tag, dtype):
 def test_a_long_request_whole_decoded_and_in_portions(tmp_path, dtype):
     """1,200 tokens: chunks of 200 and 700 positions whose edges fall into prompts, portions and decoded tokens,
     prompt attention over hundreds of keys, decoded tokens whose keys are split over several CTAs, both recurrences
-    through all of it (the linear one in segments), with graphs and without."""
+    through all of it, with graphs and without."""
     from tests.vepevik_configs import VEP_LONG as cfg
 
     ids = random_ids(cfg, 1200, 7)

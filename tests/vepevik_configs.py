@@ -111,7 +111,7 @@ VEP_D = _model(97, 100, 2e-5, [
 VEP = {"a": VEP_A, "b": VEP_B, "c": VEP_C, "d": VEP_D}
 
 # for one long request: chunks of 200 positions that begin and end in prompts and in decoded tokens, a second attention whose chunk
-# is longer than the request's first portions, prompt attention over hundreds of keys, recurrences in segments
+# is longer than the request's first portions, prompt attention over hundreds of keys, states that live through all of it
 VEP_LONG = _model(500, 256, 1e-6, [
     _layer(_att(8, 2, 64, 32, 0.25, 200, _rot(100000.0, 16), v_mix=True), _dense(96, 1.0)),
     _layer(_ret([0.875, 0.96875, 0.9921875, 0.998046875], 32, 48, _rot(10000.0, 16)), _moe(32, 8, 2, 1.5, (4, 3))),

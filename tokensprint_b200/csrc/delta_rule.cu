@@ -9,6 +9,9 @@
 // S <- diag(g) S; the decays of long portions are worked out ahead by channel_decay (every CTA of the scan that shares
 // a head reads them), those of a step of few tokens in the staging pass.
 //
+// The kernels also run the plain linear recurrence S <- decay_h S + k v^T, o = S^T q with one constant decay per head and rotated
+// q and k (retention, ts_retention_scan): the rule without its correction (u = v), without unit lengths and write strengths.
+//
 // delta_scan takes the tokens of a portion in blocks of BT (four).  With S the state before a block, Gamma(j..i] the
 // product of the decays of tokens j+1 .. i and G_i that of all tokens of the block up to i (all per key channel),
 //
@@ -59,16 +62,27 @@ struct DrGates {
   long long ld_beta, ld_decay;
   int beta_bf16;          // element type of beta
   int raw;                // 1: decay holds the raw entries; 0: the decays themselves
+  const float2* rotation; // DR_LINEAR: [T, half] cosines and sines by which entries i and i + half of q and k turn, or null
+  int half;
 };
+
+// The recurrences these kernels know.
+#define DR_HEAD 0     // the delta rule with one decay per (token, head)
+#define DR_CHANNEL 1  // with one per (token, head, key channel)
+#define DR_LINEAR 2   // no correction (u = v), q and k as they come but rotated, one constant decay per head (retention)
 
 // The block's sums over the key channels, in the order nk_0.. (squares of k), nq_0.., A_10, A_20, A_21, .., B_00, B_10, B_11, ..
 __host__ __device__ constexpr int dr_sums(int bt) { return 2 * bt + bt * bt; }
 
-// Adds up v[0 .. N) over the lanes of a warp; lane l gets the total of v[l] (N <= 32).
+// Adds up v[0 .. N) over the lanes of a warp; lane l gets the total of v[l] (N <= 32; for N <= 16 of v[l % 16]).
 template <int N>
 __device__ __forceinline__ float dr_scatter_sum(float (&v)[32], int lane) {
+  if (N <= 16) {
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
+    for (int i = 0; i < N; ++i) v[i] += __shfl_xor_sync(0xffffffffu, v[i], 16);
+  }
+#pragma unroll
+  for (int o = N <= 16 ? 8 : 16; o > 0; o >>= 1) {
     const bool up = (lane & o) != 0;
 #pragma unroll
     for (int i = 0; i < o; ++i) {
@@ -80,13 +94,13 @@ __device__ __forceinline__ float dr_scatter_sum(float (&v)[32], int lane) {
 }
 
 // M fours of key channels per thread, R lanes per value column (4 M R >= d), blocks of BT tokens.
-// CHANNEL: a decay per key channel (rows of S) instead of one per head.
-template <int M, int R, int BT, bool CHANNEL>
+template <int M, int R, int BT, int KIND, typename TX>
 __global__ void __launch_bounds__(DR_THREADS) delta_scan_kernel(
-    const float* __restrict__ x, long long ld, int q_off, int k_off, int v_off, DrGates gates, float* __restrict__ state, long long slot_stride,
+    const TX* __restrict__ x, long long ld, int q_off, int k_off, int v_off, DrGates gates, float* __restrict__ state, long long slot_stride,
     const int* __restrict__ state_slots, const int* __restrict__ cu_seqlens, float* __restrict__ out, int H, int G, int d, int e,
     float q_scale, float unit_eps, int vec) {
   ts_pdl_prologue();
+  constexpr bool CHANNEL = KIND == DR_CHANNEL, LINEAR = KIND == DR_LINEAR;
   constexpr int COLS = DR_THREADS / R;  // value columns of this CTA
   constexpr int DPAD = 4 * M * R;
   constexpr int TB = dr_round_tokens(DPAD, BT);
@@ -141,9 +155,17 @@ __global__ void __launch_bounds__(DR_THREADS) delta_scan_kernel(
     for (int u = 0; u < PF; ++u) {
       const int i = tid + u * DR_THREADS, tt = i / DPAD, c = i - tt * DPAD;
       const bool ok = tt < nt && c < d;
-      const float* row = x + (size_t)(t0 + (ok ? tt : 0)) * ld + hk * d + (ok ? c : 0);
-      pq[u] = ok ? row[q_off] : 0.f;
-      pk[u] = ok ? row[k_off] : 0.f;
+      const TX* row = x + (size_t)(t0 + (ok ? tt : 0)) * ld + hk * d + (ok ? c : 0);
+      pq[u] = ok ? ts_to_float(row[q_off]) : 0.f;
+      pk[u] = ok ? ts_to_float(row[k_off]) : 0.f;
+      if (LINEAR && ok && c < 2 * gates.half) {  // entry c turns with its partner half a rotated width away
+        const bool low = c < gates.half;
+        const int other = low ? gates.half : -gates.half;
+        const float2 cs = gates.rotation[(size_t)(t0 + tt) * gates.half + (low ? c : c - gates.half)];
+        const float sn = low ? -cs.y : cs.y;
+        pq[u] = pq[u] * cs.x + ts_to_float(row[q_off + other]) * sn;
+        pk[u] = pk[u] * cs.x + ts_to_float(row[k_off + other]) * sn;
+      }
       if (CHANNEL) pg[u] = ok ? gates.decay[(size_t)(t0 + tt) * gates.ld_decay + (size_t)h * d + c] : 1.f;
     }
 #pragma unroll
@@ -151,11 +173,11 @@ __global__ void __launch_bounds__(DR_THREADS) delta_scan_kernel(
       const int i = tid + u * DR_THREADS, tt = i / COLS, c = i - tt * COLS;
       const int vc = blockIdx.z * COLS + c;
       const bool ok = tt < nt && vc < e;
-      pv[u] = ok ? x[(size_t)(t0 + tt) * ld + v_off + h * e + vc] : 0.f;
+      pv[u] = ok ? ts_to_float(x[(size_t)(t0 + tt) * ld + v_off + h * e + vc]) : 0.f;
     }
     if (tid < nt) {
       const size_t at = (size_t)(t0 + tid) * gates.ld_beta + h;
-      pb = gates.beta_bf16 ? __bfloat162float(((const __nv_bfloat16*)gates.beta)[at]) : ((const float*)gates.beta)[at];
+      if (!LINEAR) pb = gates.beta_bf16 ? __bfloat162float(((const __nv_bfloat16*)gates.beta)[at]) : ((const float*)gates.beta)[at];
       if (!CHANNEL) pa = gates.decay[(size_t)(t0 + tid) * gates.ld_decay + h];
     }
   };
@@ -182,7 +204,7 @@ __global__ void __launch_bounds__(DR_THREADS) delta_scan_kernel(
       if (i < TB * COLS) vs[i] = pv[u];
     }
     if (tid < TB) {
-      bs[tid] = tid < nt ? 1.f / (1.f + expf(-pb)) : 0.f;
+      bs[tid] = tid >= nt ? 0.f : LINEAR ? 1.f : 1.f / (1.f + expf(-pb));
       if (!CHANNEL) g1[tid] = tid >= nt ? 1.f : gates.raw ? dr_decay(pa, bias_h, decay_rate) : pa;
     }
     __syncthreads();
@@ -234,7 +256,7 @@ __global__ void __launch_bounds__(DR_THREADS) delta_scan_kernel(
         }
       }
       // lanes 0 .. BT - 1: the factor of k_i, the next BT: of q_i; the others: their entry of A or B times the factors of its rows
-      const float own = (lane < BT ? 1.f : q_scale) / sqrtf(lane < 2 * BT ? total + unit_eps : 1.f);
+      const float own = (lane < BT ? 1.f : q_scale) / sqrtf(!LINEAR && lane < 2 * BT ? total + unit_eps : 1.f);
       int i = 0, j = 0;
       bool of_q = false;
 #pragma unroll
@@ -285,17 +307,24 @@ __global__ void __launch_bounds__(DR_THREADS) delta_scan_kernel(
       for (int m = 0; m < M; ++m)
 #pragma unroll
         for (int i = 0; i < BT; ++i) {
-          const float4 kv = k4[i * (DPAD / 4) + R * m], qv = q4[i * (DPAD / 4) + R * m];
-          sk[i] = fmaf(S[4 * m + 0], kv.x, sk[i]), sq[i] = fmaf(S[4 * m + 0], qv.x, sq[i]);
-          sk[i] = fmaf(S[4 * m + 1], kv.y, sk[i]), sq[i] = fmaf(S[4 * m + 1], qv.y, sq[i]);
-          sk[i] = fmaf(S[4 * m + 2], kv.z, sk[i]), sq[i] = fmaf(S[4 * m + 2], qv.z, sq[i]);
-          sk[i] = fmaf(S[4 * m + 3], kv.w, sk[i]), sq[i] = fmaf(S[4 * m + 3], qv.w, sq[i]);
+          const float4 qv = q4[i * (DPAD / 4) + R * m];
+          sq[i] = fmaf(S[4 * m + 0], qv.x, sq[i]);
+          sq[i] = fmaf(S[4 * m + 1], qv.y, sq[i]);
+          sq[i] = fmaf(S[4 * m + 2], qv.z, sq[i]);
+          sq[i] = fmaf(S[4 * m + 3], qv.w, sq[i]);
+          if (!LINEAR) {
+            const float4 kv = k4[i * (DPAD / 4) + R * m];
+            sk[i] = fmaf(S[4 * m + 0], kv.x, sk[i]);
+            sk[i] = fmaf(S[4 * m + 1], kv.y, sk[i]);
+            sk[i] = fmaf(S[4 * m + 2], kv.z, sk[i]);
+            sk[i] = fmaf(S[4 * m + 3], kv.w, sk[i]);
+          }
         }
 #pragma unroll
       for (int o = R >> 1; o > 0; o >>= 1)
 #pragma unroll
         for (int i = 0; i < BT; ++i) {
-          sk[i] += __shfl_xor_sync(0xffffffffu, sk[i], o);
+          if (!LINEAR) sk[i] += __shfl_xor_sync(0xffffffffu, sk[i], o);
           sq[i] += __shfl_xor_sync(0xffffffffu, sq[i], o);
         }
       float u[BT];
@@ -303,7 +332,7 @@ __global__ void __launch_bounds__(DR_THREADS) delta_scan_kernel(
       for (int i = 0; i < BT; ++i) {
         float rest = vs[(blk * BT + i) * COLS + cl] - sk[i];
 #pragma unroll
-        for (int j = 0; j < i; ++j) rest = fmaf(-coef[blk][i * (i - 1) / 2 + j], u[j], rest);
+        for (int j = 0; j < (LINEAR ? 0 : i); ++j) rest = fmaf(-coef[blk][i * (i - 1) / 2 + j], u[j], rest);
         u[i] = bs[blk * BT + i] * rest;
       }
 #pragma unroll
@@ -348,15 +377,15 @@ __global__ void __launch_bounds__(DR_THREADS) delta_scan_kernel(
   }
 }
 
-template <int M, int R, int BT, bool CHANNEL>
-static int dr_launch(const float* x, long long ld, int q_off, int k_off, int v_off, const DrGates& gates, float* state, long long slot_stride,
+template <int M, int R, int BT, int KIND, typename TX>
+static int dr_launch(const TX* x, long long ld, int q_off, int k_off, int v_off, const DrGates& gates, float* state, long long slot_stride,
                      const int* state_slots, const int* cu_seqlens, float* out, int B, int H, int G, int d, int e, float q_scale, float unit_eps,
                      cudaStream_t s) {
   constexpr int COLS = DR_THREADS / R;
   const dim3 grid(B, H, (e + COLS - 1) / COLS);
   if (grid.z > 65535) return TS_ERR_UNSUPPORTED_SIZE;
   const int vec = d % 4 == 0 && slot_stride % 4 == 0 && (uintptr_t)state % 16 == 0;
-  return ts_launch(delta_scan_kernel<M, R, BT, CHANNEL>, grid, dim3(DR_THREADS), 0, s, x, ld, q_off, k_off, v_off, gates, state, slot_stride,
+  return ts_launch(delta_scan_kernel<M, R, BT, KIND, TX>, grid, dim3(DR_THREADS), 0, s, x, ld, q_off, k_off, v_off, gates, state, slot_stride,
                    state_slots, cu_seqlens, out, H, G, d, e, q_scale, unit_eps, vec);
 }
 
@@ -403,16 +432,18 @@ __device__ __forceinline__ float dp_scatter(float (&v)[N], int r) {
   return t;
 }
 
-template <int M, int R, int CT, int CPT, bool CHANNEL>
+template <int M, int R, int CT, int CPT, int KIND, typename TX>
 __global__ void __launch_bounds__(CT + 128, 2) delta_portion_kernel(
-    const float* __restrict__ x, long long ld, int q_off, int k_off, int v_off, DrGates gates, float* __restrict__ state, long long slot_stride,
+    const TX* __restrict__ x, long long ld, int q_off, int k_off, int v_off, DrGates gates, float* __restrict__ state, long long slot_stride,
     const int* __restrict__ state_slots, const int* __restrict__ cu_seqlens, float* __restrict__ out, int H, int G, int d, int e,
     float q_scale, float unit_eps, int vec) {
   ts_pdl_prologue();
+  constexpr bool CHANNEL = KIND == DR_CHANNEL, LINEAR = KIND == DR_LINEAR;
   using Buffer = DpBuffer<M, R, CT, CPT>;
   constexpr int COLS = Buffer::COLS, DPAD = Buffer::DPAD, BT = DP_BT, TB = DP_NB * BT;
-  constexpr int NCH = (DPAD + 31) / 32, NV = (BT * COLS + 31) / 32;  // channels and values per preparing lane and block
-  constexpr int NA = BT * (BT - 1) / 2, NS = dr_sums(BT);
+  // (LINEAR: an even number of channels, so that the two of a rotated pair sit in one lane)
+  constexpr int NCH = LINEAR && DPAD <= 32 ? 2 : (DPAD + 31) / 32, NV = (BT * COLS + 31) / 32;  // channels and values per preparing lane and block
+  constexpr int NA = BT * (BT - 1) / 2, NS = dr_sums(BT), SA = 2 * BT + NA, SB = LINEAR ? 0 : SA;  // SB: where B begins among the sums
   extern __shared__ __align__(16) unsigned char dp_smem[];
   Buffer* const buffers = reinterpret_cast<Buffer*>(dp_smem);
   const int b = blockIdx.x, h = blockIdx.y;
@@ -450,11 +481,12 @@ __global__ void __launch_bounds__(CT + 128, 2) delta_portion_kernel(
         }
     }
   }
-  constexpr int NVAL = 2 * BT * CPT;       // sums of a block: for every column S^T k~ of the four tokens, then S^T q~
+  constexpr int KD = LINEAR ? 0 : BT;       // sums of a block: for every column S^T k~ of the four tokens (not LINEAR), then S^T q~
+  constexpr int NC = KD + BT, NVAL = NC * CPT;
   constexpr bool SCATTER = R >= NVAL;
   constexpr int SHARE = SCATTER ? R / NVAL : 1;
   // the column and token whose read-out this lane writes (SCATTER)
-  const int w_idx = r / SHARE, w_p = w_idx / (2 * BT), w_i = w_idx % (2 * BT) - BT;
+  const int w_idx = r / SHARE, w_p = w_idx / NC, w_i = w_idx % NC - KD;
   bool writes = false;
   int w_col = col0;
 #pragma unroll
@@ -479,14 +511,21 @@ __global__ void __launch_bounds__(CT + 128, 2) delta_portion_kernel(
       for (int m = 0; m < M; ++m)
 #pragma unroll
         for (int i = 0; i < BT; ++i) {
-          const float4 kv = k4[i * (DPAD / 4) + R * m], qv = q4[i * (DPAD / 4) + R * m];
+          const float4 qv = q4[i * (DPAD / 4) + R * m];
+          const float4 kv = LINEAR ? qv : k4[i * (DPAD / 4) + R * m];
 #pragma unroll
           for (int p = 0; p < CPT; ++p) {
-            float &a = sums[p * 2 * BT + i], &z = sums[p * 2 * BT + BT + i];
-            a = fmaf(S[p][4 * m + 0], kv.x, a), z = fmaf(S[p][4 * m + 0], qv.x, z);
-            a = fmaf(S[p][4 * m + 1], kv.y, a), z = fmaf(S[p][4 * m + 1], qv.y, z);
-            a = fmaf(S[p][4 * m + 2], kv.z, a), z = fmaf(S[p][4 * m + 2], qv.z, z);
-            a = fmaf(S[p][4 * m + 3], kv.w, a), z = fmaf(S[p][4 * m + 3], qv.w, z);
+            float &a = sums[p * NC + i], &z = sums[p * NC + KD + i];
+            if (!LINEAR) {
+              a = fmaf(S[p][4 * m + 0], kv.x, a);
+              a = fmaf(S[p][4 * m + 1], kv.y, a);
+              a = fmaf(S[p][4 * m + 2], kv.z, a);
+              a = fmaf(S[p][4 * m + 3], kv.w, a);
+            }
+            z = fmaf(S[p][4 * m + 0], qv.x, z);
+            z = fmaf(S[p][4 * m + 1], qv.y, z);
+            z = fmaf(S[p][4 * m + 2], qv.z, z);
+            z = fmaf(S[p][4 * m + 3], qv.w, z);
           }
         }
       const float4 bb = buf.beta[blk], c0 = buf.coef[blk][0], c1 = buf.coef[blk][1], c2 = buf.coef[blk][2], c3 = buf.coef[blk][3];
@@ -505,15 +544,19 @@ __global__ void __launch_bounds__(CT + 128, 2) delta_portion_kernel(
         const float4 vv = buf.v[blk][cl + p * (COLS / CPT)];
         float sk[BT];
 #pragma unroll
-        for (int i = 0; i < BT; ++i) sk[i] = SCATTER ? __shfl_sync(0xffffffffu, mine, (p * 2 * BT + i) * SHARE, R) : sums[p * 2 * BT + i];
-        u[p][0] = bb.x * (vv.x - sk[0]);
-        u[p][1] = bb.y * fmaf(-c0.x, u[p][0], vv.y - sk[1]);
-        u[p][2] = bb.z * fmaf(-c0.z, u[p][1], fmaf(-c0.y, u[p][0], vv.z - sk[2]));
-        u[p][3] = bb.w * fmaf(-c1.y, u[p][2], fmaf(-c1.x, u[p][1], fmaf(-c0.w, u[p][0], vv.w - sk[3])));
+        for (int i = 0; i < BT; ++i) sk[i] = LINEAR ? 0.f : SCATTER ? __shfl_sync(0xffffffffu, mine, (p * NC + i) * SHARE, R) : sums[p * NC + i];
+        if (LINEAR) {
+          u[p][0] = vv.x, u[p][1] = vv.y, u[p][2] = vv.z, u[p][3] = vv.w;
+        } else {
+          u[p][0] = bb.x * (vv.x - sk[0]);
+          u[p][1] = bb.y * fmaf(-c0.x, u[p][0], vv.y - sk[1]);
+          u[p][2] = bb.z * fmaf(-c0.z, u[p][1], fmaf(-c0.y, u[p][0], vv.z - sk[2]));
+          u[p][3] = bb.w * fmaf(-c1.y, u[p][2], fmaf(-c1.x, u[p][1], fmaf(-c0.w, u[p][0], vv.w - sk[3])));
+        }
       }
 #pragma unroll
       for (int m = 0; m < M; ++m) {
-        const float4 gv = g4[R * m];
+        const float4 gv = LINEAR ? make_float4(c0.x, c0.x, c0.x, c0.x) : g4[R * m];
         const float4 a = e4[R * m], f = e4[(DPAD / 4) + R * m], q = e4[2 * (DPAD / 4) + R * m], w = e4[3 * (DPAD / 4) + R * m];
 #pragma unroll
         for (int p = 0; p < CPT; ++p) {
@@ -542,7 +585,7 @@ __global__ void __launch_bounds__(CT + 128, 2) delta_portion_kernel(
 #pragma unroll
           for (int i = 0; i < BT; ++i)
             if (live[p] && i % R == r && blk * BT + i < nt)
-              out[(size_t)(t_begin + t0 + blk * BT + i) * out_row + (size_t)h * e + col0 + cl + p * (COLS / CPT)] = sums[p * 2 * BT + BT + i] + reads(u[p], i);
+              out[(size_t)(t_begin + t0 + blk * BT + i) * out_row + (size_t)h * e + col0 + cl + p * (COLS / CPT)] = sums[p * NC + KD + i] + reads(u[p], i);
       }
     }
   };
@@ -551,21 +594,32 @@ __global__ void __launch_bounds__(CT + 128, 2) delta_portion_kernel(
   const int blk = warp - CT / 32;
   const int hk = h / (H / G);
   const float decay_rate = gates.raw ? expf(gates.a_log[h]) : 0.f;
-  float q[NCH][BT], k[NCH][BT], g[CHANNEL ? NCH : 1][BT], v[NV], pb = 0.f;
+  // (what is fetched stays as it came until it is used: a conversion would wait for the load)
+  TX fq[NCH][BT], fk[NCH][BT], fv[NV];
+  float g[CHANNEL ? NCH : 1][BT], pb = 0.f;
+  float2 turn[LINEAR ? NCH / 2 : 1][BT];
+  // the key channel of a lane's entry n2: lane + 32 n2, or (LINEAR) such that entries 2 m and 2 m + 1 are a rotated pair while there
+  // are any left, then the channels behind the rotated ones
+  auto channel = [&](int n2) {
+    if (!LINEAR) return lane + 32 * n2;
+    const int pair = lane + 32 * (n2 >> 1);
+    return pair < gates.half ? pair + (n2 & 1) * gates.half : 2 * pair + (n2 & 1);
+  };
   auto fetch = [&](int n) {
     const int t0 = t_begin + n * TB + blk * BT;
     // a token beyond the portion's end writes nothing into the state: k = 0, beta = 0, decay 1
 #pragma unroll
     for (int i = 0; i < BT; ++i) {
       const bool there = t0 + i < t_end;
-      const float* row = x + (size_t)(there ? t0 + i : t_begin) * ld + hk * d;
+      const TX* row = x + (size_t)(there ? t0 + i : t_begin) * ld + hk * d;
       const float* drow = gates.decay + (size_t)(there ? t0 + i : t_begin) * gates.ld_decay + (CHANNEL ? (size_t)h * d : h);
 #pragma unroll
       for (int n2 = 0; n2 < NCH; ++n2) {
-        const int c = lane + 32 * n2;
+        const int c = channel(n2);
         const bool ok = there && c < d;
-        q[n2][i] = ok ? row[q_off + c] : 0.f;
-        k[n2][i] = ok ? row[k_off + c] : 0.f;
+        fq[n2][i] = ok ? row[q_off + c] : TX(0.f);
+        fk[n2][i] = ok ? row[k_off + c] : TX(0.f);
+        if (LINEAR && n2 % 2 == 0) turn[n2 / 2][i] = ok && c < gates.half ? gates.rotation[(size_t)(t0 + i) * gates.half + c] : make_float2(1.f, 0.f);
         if (CHANNEL) g[n2][i] = ok ? drow[c] : 1.f;
       }
       if (!CHANNEL) g[0][i] = there ? drow[0] : 1.f;
@@ -573,9 +627,9 @@ __global__ void __launch_bounds__(CT + 128, 2) delta_portion_kernel(
 #pragma unroll
     for (int n2 = 0; n2 < NV; ++n2) {
       const int at = lane + 32 * n2, i = at / COLS, c = at % COLS;
-      v[n2] = at < BT * COLS && t0 + i < t_end && col0 + c < e ? x[(size_t)(t0 + i) * ld + v_off + h * e + col0 + c] : 0.f;
+      fv[n2] = at < BT * COLS && t0 + i < t_end && col0 + c < e ? x[(size_t)(t0 + i) * ld + v_off + h * e + col0 + c] : TX(0.f);
     }
-    if (lane < BT && t0 + lane < t_end) {
+    if (!LINEAR && lane < BT && t0 + lane < t_end) {
       const size_t at = (size_t)(t0 + lane) * gates.ld_beta + h;
       pb = gates.beta_bf16 ? __bfloat162float(((const __nv_bfloat16*)gates.beta)[at]) : ((const float*)gates.beta)[at];
     }
@@ -594,6 +648,22 @@ __global__ void __launch_bounds__(CT + 128, 2) delta_portion_kernel(
           if (t0 + i < t_end && (!CHANNEL || c < d)) g[n2][i] = dr_decay(g[n2][i], bias, decay_rate);
       }
     }
+    float q[NCH][BT], k[NCH][BT];
+#pragma unroll
+    for (int n2 = 0; n2 < NCH; ++n2)
+#pragma unroll
+      for (int i = 0; i < BT; ++i) q[n2][i] = ts_to_float(fq[n2][i]), k[n2][i] = ts_to_float(fk[n2][i]);
+    if (LINEAR && gates.half > 0) {
+#pragma unroll
+      for (int n2 = 0; n2 + 1 < NCH; n2 += 2)
+#pragma unroll
+        for (int i = 0; i < BT; ++i) {
+          const float2 cs = turn[LINEAR ? n2 / 2 : 0][i];
+          const float qu = q[n2][i], ku = k[n2][i];
+          q[n2][i] = qu * cs.x - q[n2 + 1][i] * cs.y, q[n2 + 1][i] = q[n2 + 1][i] * cs.x + qu * cs.y;
+          k[n2][i] = ku * cs.x - k[n2 + 1][i] * cs.y, k[n2 + 1][i] = k[n2 + 1][i] * cs.x + ku * cs.y;
+        }
+    }
     float sum[32];
 #pragma unroll
     for (int i = 0; i < 32; ++i) sum[i] = 0.f;
@@ -602,6 +672,7 @@ __global__ void __launch_bounds__(CT + 128, 2) delta_portion_kernel(
       const float (&gt)[BT] = g[CHANNEL ? n2 : 0];
 #pragma unroll
       for (int i = 0; i < BT; ++i) {
+        if (LINEAR) continue;
         sum[i] = fmaf(k[n2][i], k[n2][i], sum[i]);
         sum[BT + i] = fmaf(q[n2][i], q[n2][i], sum[BT + i]);
       }
@@ -612,20 +683,20 @@ __global__ void __launch_bounds__(CT + 128, 2) delta_portion_kernel(
         for (int i = j; i < BT; ++i) {
           if (i > j) {
             w *= gt[i];
-            sum[2 * BT + i * (i - 1) / 2 + j] = fmaf(k[n2][i], w, sum[2 * BT + i * (i - 1) / 2 + j]);
+            if (!LINEAR) sum[2 * BT + i * (i - 1) / 2 + j] = fmaf(k[n2][i], w, sum[2 * BT + i * (i - 1) / 2 + j]);
           }
-          sum[2 * BT + NA + i * (i + 1) / 2 + j] = fmaf(q[n2][i], w, sum[2 * BT + NA + i * (i + 1) / 2 + j]);
+          sum[SB + i * (i + 1) / 2 + j] = fmaf(q[n2][i], w, sum[SB + i * (i + 1) / 2 + j]);
         }
       }
     }
-    const float total = dr_scatter_sum<NS>(sum, lane);
+    const float total = dr_scatter_sum<LINEAR ? NS - SA : NS>(sum, lane);
     // lanes 0 .. 3: the factor of k_i, 4 .. 7: of q_i; the others: their entry of A or B times the factors of its rows
     const float own = (lane < BT ? 1.f : q_scale) / sqrtf(lane < 2 * BT ? total + unit_eps : 1.f);
     float mk[BT], mq[BT];
 #pragma unroll
     for (int i = 0; i < BT; ++i) {
-      mk[i] = __shfl_sync(0xffffffffu, own, i);
-      mq[i] = __shfl_sync(0xffffffffu, own, BT + i);
+      mk[i] = LINEAR ? 1.f : __shfl_sync(0xffffffffu, own, i);
+      mq[i] = LINEAR ? q_scale : __shfl_sync(0xffffffffu, own, BT + i);
     }
     float f = 0.f;
 #pragma unroll
@@ -635,22 +706,27 @@ __global__ void __launch_bounds__(CT + 128, 2) delta_portion_kernel(
         if (j < i && lane == 2 * BT + i * (i - 1) / 2 + j) f = mk[i] * mk[j];
         if (lane == 2 * BT + NA + i * (i + 1) / 2 + j) f = mq[i] * mk[j];
       }
-    if (lane >= 2 * BT && lane < NS) reinterpret_cast<float*>(buf.coef[blk])[lane - 2 * BT] = total * f;
-    if (lane < BT) reinterpret_cast<float*>(&buf.beta[blk])[lane] = t0 + lane < t_end ? 1.f / (1.f + expf(-pb)) : 0.f;
+    if (LINEAR) {  // no A: its first place takes the block's decay
+      if (lane < NS - SA) reinterpret_cast<float*>(buf.coef[blk])[NA + lane] = total * q_scale;
+      if (lane == 16) buf.coef[blk][0].x = g[0][0] * g[0][1] * g[0][2] * g[0][3];
+    } else if (lane >= 2 * BT && lane < NS) {
+      reinterpret_cast<float*>(buf.coef[blk])[lane - 2 * BT] = total * f;
+    }
+    if (!LINEAR && lane < BT) reinterpret_cast<float*>(&buf.beta[blk])[lane] = t0 + lane < t_end ? 1.f / (1.f + expf(-pb)) : 0.f;
 #pragma unroll
     for (int n2 = 0; n2 < NCH; ++n2) {
-      const int c = lane + 32 * n2;
+      const int c = channel(n2);
       const float (&gt)[BT] = g[CHANNEL ? n2 : 0];
-      if (DPAD % 32 == 0 || c < DPAD) {
+      if ((DPAD % 32 == 0 && !LINEAR) || c < DPAD) {
         float w = 1.f, back = 1.f;
 #pragma unroll
         for (int i = 0; i < BT; ++i) {
           w *= gt[i];
           k[n2][i] *= mk[i];
-          buf.kt[blk][i][c] = k[n2][i] * w;
+          if (!LINEAR) buf.kt[blk][i][c] = k[n2][i] * w;
           buf.qt[blk][i][c] = q[n2][i] * mq[i] * w;
         }
-        buf.ge[blk][c] = w;
+        if (!LINEAR) buf.ge[blk][c] = w;
 #pragma unroll
         for (int i = BT - 1; i >= 0; --i) {
           buf.ke[blk][i][c] = k[n2][i] * back;
@@ -661,7 +737,7 @@ __global__ void __launch_bounds__(CT + 128, 2) delta_portion_kernel(
 #pragma unroll
     for (int n2 = 0; n2 < NV; ++n2) {
       const int at = lane + 32 * n2, i = at / COLS, c = at % COLS;
-      if (at < BT * COLS) reinterpret_cast<float*>(&buf.v[blk][c])[i] = v[n2];
+      if (at < BT * COLS) reinterpret_cast<float*>(&buf.v[blk][c])[i] = ts_to_float(fv[n2]);
     }
   };
 
@@ -701,8 +777,8 @@ __global__ void __launch_bounds__(CT + 128, 2) delta_portion_kernel(
   }
 }
 
-template <int M, int R, int CT, int CPT, bool CHANNEL>
-static int dp_launch(const float* x, long long ld, int q_off, int k_off, int v_off, const DrGates& gates, float* state, long long slot_stride,
+template <int M, int R, int CT, int CPT, int KIND, typename TX>
+static int dp_launch(const TX* x, long long ld, int q_off, int k_off, int v_off, const DrGates& gates, float* state, long long slot_stride,
                      const int* state_slots, const int* cu_seqlens, float* out, int B, int H, int G, int d, int e, float q_scale, float unit_eps,
                      cudaStream_t s) {
   constexpr int COLS = CT / R * CPT;
@@ -711,24 +787,24 @@ static int dp_launch(const float* x, long long ld, int q_off, int k_off, int v_o
   if (grid.z > 65535) return TS_ERR_UNSUPPORTED_SIZE;
   static bool sized = false;
   if (smem > 48 * 1024 && !sized) {
-    const cudaError_t err = cudaFuncSetAttribute(delta_portion_kernel<M, R, CT, CPT, CHANNEL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const cudaError_t err = cudaFuncSetAttribute(delta_portion_kernel<M, R, CT, CPT, KIND, TX>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (err != cudaSuccess) return (int)err;
     sized = true;
   }
   const int vec = d % 4 == 0 && slot_stride % 4 == 0 && (uintptr_t)state % 16 == 0;
-  return ts_launch(delta_portion_kernel<M, R, CT, CPT, CHANNEL>, grid, dim3(CT + 128), smem, s, x, ld, q_off, k_off, v_off, gates, state, slot_stride,
+  return ts_launch(delta_portion_kernel<M, R, CT, CPT, KIND, TX>, grid, dim3(CT + 128), smem, s, x, ld, q_off, k_off, v_off, gates, state, slot_stride,
                    state_slots, cu_seqlens, out, H, G, d, e, q_scale, unit_eps, vec);
 }
 
 // How the state of one head is cut over threads for key width d: in portions a thread holds 4 or 8 key channels of two value
 // columns (of one for narrow keys, in steps of one token 16 channels of one; more where a warp's lanes would not do), and as many
 // lanes share a column as that takes: a function of d alone.
-template <bool CHANNEL>
-static int dr_dispatch(const float* x, long long ld, int q_off, int k_off, int v_off, const DrGates& gates, float* state, long long slot_stride,
+template <int KIND, typename TX>
+static int dr_dispatch(const TX* x, long long ld, int q_off, int k_off, int v_off, const DrGates& gates, float* state, long long slot_stride,
                        const int* state_slots, const int* cu_seqlens, float* out, int B, int H, int G, int d, int e, float q_scale,
                        float unit_eps, int single, cudaStream_t s) {
 #define DR_GO(MM, RR, BB) \
-  return dr_launch<MM, RR, BB, CHANNEL>(x, ld, q_off, k_off, v_off, gates, state, slot_stride, state_slots, cu_seqlens, out, B, H, G, d, e, q_scale, unit_eps, s)
+  return dr_launch<MM, RR, BB, KIND, TX>(x, ld, q_off, k_off, v_off, gates, state, slot_stride, state_slots, cu_seqlens, out, B, H, G, d, e, q_scale, unit_eps, s)
   if (single) {
     if (d <= 4) DR_GO(1, 1, 1);
     if (d <= 8) DR_GO(2, 1, 1);
@@ -741,7 +817,7 @@ static int dr_dispatch(const float* x, long long ld, int q_off, int k_off, int v
     DR_GO(8, 32, 1);
   }
 #define DP_GO(MM, RR, CC, PP) \
-  return dp_launch<MM, RR, CC, PP, CHANNEL>(x, ld, q_off, k_off, v_off, gates, state, slot_stride, state_slots, cu_seqlens, out, B, H, G, d, e, q_scale, unit_eps, s)
+  return dp_launch<MM, RR, CC, PP, KIND, TX>(x, ld, q_off, k_off, v_off, gates, state, slot_stride, state_slots, cu_seqlens, out, B, H, G, d, e, q_scale, unit_eps, s)
   if (d <= 8) DP_GO(2, 1, 128, 1);
   if (d <= 16) DP_GO(2, 2, 128, 1);
   if (d <= 32) DP_GO(1, 8, 128, 1);
@@ -767,10 +843,30 @@ TS_EXPORT int ts_delta_scan(const float* x, long long ld, int q_off, int k_off, 
     return TS_ERR_BAD_ARGUMENT;
   if (d > DR_MAX_KEY_DIM || B > 65535 * 16 || H > 65535) return TS_ERR_UNSUPPORTED_SIZE;
   cudaStream_t s = (cudaStream_t)stream;
-  const DrGates gates = {beta, decay, a_log, dt_bias, ld_beta, ld_decay, beta_dtype == TS_DTYPE_BF16 ? 1 : 0, raw};
+  const DrGates gates = {beta, decay, a_log, dt_bias, ld_beta, ld_decay, beta_dtype == TS_DTYPE_BF16 ? 1 : 0, raw, nullptr, 0};
   if (per_channel)
-    return dr_dispatch<true>(x, ld, q_off, k_off, v_off, gates, state, slot_stride, state_slots, cu_seqlens, out, B, H, G, d, e, q_scale, unit_eps, single, s);
-  return dr_dispatch<false>(x, ld, q_off, k_off, v_off, gates, state, slot_stride, state_slots, cu_seqlens, out, B, H, G, d, e, q_scale, unit_eps, single, s);
+    return dr_dispatch<DR_CHANNEL, float>(x, ld, q_off, k_off, v_off, gates, state, slot_stride, state_slots, cu_seqlens, out, B, H, G, d, e, q_scale, unit_eps, single, s);
+  return dr_dispatch<DR_HEAD, float>(x, ld, q_off, k_off, v_off, gates, state, slot_stride, state_slots, cu_seqlens, out, B, H, G, d, e, q_scale, unit_eps, single, s);
+}
+
+// Retention: S <- decay_h S + k v^T, o = q_scale S^T q per head, with q, k, v columns of x [T, ..] of the compute type, q and k
+// rotated as they are read (rotation [T, half, 2] cosines and sines, entry i < half with entry i + half; half = 0: not).
+TS_EXPORT int ts_retention_scan(const void* x, int dtype, long long ld, int q_off, int k_off, int v_off, const float* rotation, int half,
+                                const float* decay, float* state, long long slot_stride, const int* state_slots, const int* cu_seqlens,
+                                float* out, int B, int H, int G, int d, int e, float q_scale, int single, void* stream) {
+  if (B <= 0) return 0;
+  if (H <= 0 || G <= 0 || H % G || d <= 0 || e <= 0 || decay == nullptr || half < 0 || 2 * half > d || (half > 0 && rotation == nullptr))
+    return TS_ERR_BAD_ARGUMENT;
+  if (d > DR_MAX_KEY_DIM || B > 65535 * 16 || H > 65535) return TS_ERR_UNSUPPORTED_SIZE;
+  cudaStream_t s = (cudaStream_t)stream;
+  const DrGates gates = {nullptr, decay, nullptr, nullptr, 0, 0, 0, 0, reinterpret_cast<const float2*>(rotation), half};
+  if (dtype == TS_DTYPE_F32)
+    return dr_dispatch<DR_LINEAR, float>((const float*)x, ld, q_off, k_off, v_off, gates, state, slot_stride, state_slots, cu_seqlens, out, B, H, G, d, e,
+                                         q_scale, 0.f, single, s);
+  if (dtype == TS_DTYPE_BF16)
+    return dr_dispatch<DR_LINEAR, __nv_bfloat16>((const __nv_bfloat16*)x, ld, q_off, k_off, v_off, gates, state, slot_stride, state_slots, cu_seqlens,
+                                                 out, B, H, G, d, e, q_scale, 0.f, single, s);
+  return TS_ERR_BAD_ARGUMENT;
 }
 
 // z[t, h * d + c] <- exp(-exp(a_log[h]) softplus(z[t, h * d + c] + dt_bias[h * d + c])), in place, float32.

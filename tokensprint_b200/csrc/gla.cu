@@ -155,7 +155,7 @@ __global__ void __launch_bounds__(GLA_THREADS, GLA_MIN_BLOCKS) gla_scan_kernel(
         const size_t at = (size_t)tr * ld_qkv + qk_off + cr;
         fq[j] = gla_load(q + at);
         fk[j] = gla_load(k + at);
-        fa[j] = decay_scalar == 2 ? gla_load(decay + h) : decay_scalar ? gla_load(decay + (size_t)tr * H + h) : gla_load(decay + (size_t)tr * Hd + a_off + cr);
+        fa[j] = decay_scalar ? gla_load(decay + (size_t)tr * H + h) : gla_load(decay + (size_t)tr * Hd + a_off + cr);
         fb[j] = kscale ? gla_load(kscale + (size_t)tr * H + h) : 1.f;
       }
       tt += step_t, c += step_c;
@@ -264,7 +264,7 @@ __global__ void __launch_bounds__(GLA_THREADS) gla_step_kernel(
     const TA* __restrict__ q, const TA* __restrict__ k, const TA* __restrict__ v, long long ld_qkv, const float* __restrict__ decay,
     float q_scale, float* __restrict__ state, const int* __restrict__ state_slots, const int* __restrict__ cu_seqlens,
     float* __restrict__ o, int H, int d, int e, int R, int cols_per_cta, const float* __restrict__ kscale, int decay_scalar, int groups,
-    int ev, long long slot_stride, const float2* __restrict__ rotation, int half) {
+    int ev, long long slot_stride) {
   ts_pdl_prologue();
   const int b = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * cols_per_cta;
   const int t = cu_seqlens[b];
@@ -278,7 +278,7 @@ __global__ void __launch_bounds__(GLA_THREADS) gla_step_kernel(
   for (int i = 0; i < KP; ++i) s_reg[i] = (has_col && CH(i) < d) ? S[(size_t)(CH(i)) * e + col] : 0.f;
   const size_t row = (size_t)t * ld_qkv, qk_off = (size_t)(h / (H / groups)) * d;
   const float scale_k = kscale ? kscale[(size_t)t * H + h] : 1.f;
-  const float a_all = decay_scalar == 2 ? decay[h] : decay_scalar ? decay[(size_t)t * H + h] : 1.f;
+  const float a_all = decay_scalar ? decay[(size_t)t * H + h] : 1.f;
   const float* a_row = decay + (size_t)t * H * d + (size_t)h * d;
   const float vv = !has_col ? 0.f : (col < ev ? ts_to_float(v[row + (size_t)h * ev + col]) : 1.f);
   float acc = 0.f;
@@ -287,17 +287,8 @@ __global__ void __launch_bounds__(GLA_THREADS) gla_step_kernel(
     const int ch = CH(i);
     if (ch < d) {
       const float a = decay_scalar ? a_all : a_row[ch];
-      float kk = ts_to_float(k[row + qk_off + ch]), qq = ts_to_float(q[row + qk_off + ch]);
-      if (ch < 2 * half) {  // channel ch turns with its partner half a rotated width away
-        const bool low = ch < half;
-        const size_t other = row + qk_off + (low ? ch + half : ch - half);
-        const float2 cs = rotation[(size_t)t * half + (low ? ch : ch - half)];
-        const float sn = low ? -cs.y : cs.y;
-        kk = kk * cs.x + ts_to_float(k[other]) * sn;
-        qq = qq * cs.x + ts_to_float(q[other]) * sn;
-      }
-      s_reg[i] = fmaf(a, s_reg[i], kk * scale_k * vv);
-      acc = fmaf(s_reg[i], qq * q_scale, acc);
+      s_reg[i] = fmaf(a, s_reg[i], ts_to_float(k[row + qk_off + ch]) * scale_k * vv);
+      acc = fmaf(s_reg[i], ts_to_float(q[row + qk_off + ch]) * q_scale, acc);
     }
   }
   for (int w = 1; w < R; w <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, w);
@@ -313,12 +304,10 @@ __global__ void __launch_bounds__(GLA_THREADS) gla_step_kernel(
 // What the general form of the recurrence has beyond gated linear attention's (see ts_linear_scan).
 struct GlaExtra {
   const float* kscale;    // [T, H] a factor on k per (token, head), or null
-  int decay_scalar;       // 1: decay is [T, H], one number per (token, head) for all key channels; 2: [H], one constant per head
+  int decay_scalar;       // 1: decay is [T, H], one number per (token, head) for all key channels
   int groups;             // q and k have `groups` heads; head h reads group h / (H / groups)
   int ev;                 // columns of v per head; the state has e >= ev columns, column ev (if any) sees the value 1
   long long slot_stride;  // floats from one request's state to the next
-  const float2* rotation; // [T, half] cosines and sines by which the first 2 half entries of q and k turn (steps of one token), or null
-  int half;
 };
 
 template <typename TA, int KP, int MODE>
@@ -370,7 +359,7 @@ static int dispatch_gla_scan(const void* q, const void* k, const void* v, long l
 #define GLA_STEP_CASE(KP) \
     if (kp1 <= KP) \
       return ts_launch(gla_step_kernel<TA, KP>, grid, dim3(GLA_THREADS), 0, s, (const TA*)q, (const TA*)k, (const TA*)v, ld_qkv, decay, q_scale, \
-                       state, state_slots, cu_seqlens, o, H, d, e, R, cols, x.kscale, x.decay_scalar, x.groups, x.ev, x.slot_stride, x.rotation, x.half)
+                       state, state_slots, cu_seqlens, o, H, d, e, R, cols, x.kscale, x.decay_scalar, x.groups, x.ev, x.slot_stride)
     GLA_STEP_CASE(4);
     GLA_STEP_CASE(8);
     GLA_STEP_CASE(12);
@@ -453,7 +442,7 @@ TS_EXPORT int ts_gla_scan(const void* q, const void* k, const void* v, long long
   if (H <= 0 || d <= 0 || e <= 0 || segs < 1 || (segs > 1 && (seg_len < 1 || scratch == nullptr))) return TS_ERR_BAD_ARGUMENT;
   if ((long long)B * segs > 0x7fffffffLL) return TS_ERR_UNSUPPORTED_SIZE;
   cudaStream_t s = (cudaStream_t)stream;
-  const GlaExtra x = {nullptr, 0, H, e, (long long)H * d * e, nullptr, 0};
+  const GlaExtra x = {nullptr, 0, H, e, (long long)H * d * e};
   if (act_dtype == TS_DTYPE_F32)
     return dispatch_gla_scan<float>(q, k, v, ld_qkv, decay, q_scale, state, state_slots, cu_seqlens, o, B, H, d, e, segs, seg_len, scratch, s, x);
   if (act_dtype == TS_DTYPE_BF16)
@@ -464,27 +453,23 @@ TS_EXPORT int ts_gla_scan(const void* q, const void* k, const void* v, long long
 
 // The same recurrence in its general form, for mixers whose decay is one number per (token, head):
 //   S_t = a_t S_(t-1) + (b_t k_t) v_t^T,   o_t = S_t^T (q_t * q_scale)
-// decay = a [T, H] float32 (`decay_scalar` = 1; 0: [T, H*d] as above; 2: [H], a constant per head); kscale = b [T, H] float32 or null;
+// decay = a [T, H] float32 (`decay_scalar` = 1; 0: [T, H*d] as above); kscale = b [T, H] float32 or null;
 // q, k [T, groups*d] (head h reads group h / (H / groups)) and v [T, H*ev], views with the common row
 // stride ld_qkv; the state of a request starts `slot_stride` floats after the one before it and holds
 // [H, d, e] with e = ev or ev + 1: a column beyond v's sees the value 1 in every token, so that it
 // carries sum_t (products of decays) b_t k_t, the normaliser of a matrix memory, and its read-out
 // n_t . q_t arrives as column ev of o [T, H*e].
-// rotation [T, half, 2] (cosine, sine), half > 0: q and k are rotated as they are read (entry i < half with entry
-// i + half); only in steps of one token per sequence (segs = seg_len = 1), longer portions bring rotated rows.
 TS_EXPORT int ts_linear_scan(const void* q, const void* k, const void* v, long long ld_qkv, int act_dtype, const float* decay,
                              int decay_scalar, const float* kscale, float q_scale, float* state, long long slot_stride, const int* state_slots,
                              const int* cu_seqlens, float* o, int B, int H, int groups, int d, int ev, int e, int segs, int seg_len,
-                             float* scratch, const float* rotation, int half, void* stream) {
+                             float* scratch, void* stream) {
   if (B <= 0) return 0;
-  if (decay_scalar < 0 || decay_scalar > 2 || half < 0 || 2 * half > d || (half > 0 && (rotation == nullptr || segs != 1 || seg_len != 1)))
-    return TS_ERR_BAD_ARGUMENT;
   if (H <= 0 || d <= 0 || ev <= 0 || (e != ev && e != ev + 1) || groups <= 0 || H % groups || segs < 1 ||
       (segs > 1 && (seg_len < 1 || scratch == nullptr)) || slot_stride < (long long)H * d * e)
     return TS_ERR_BAD_ARGUMENT;
   if ((long long)B * segs > 0x7fffffffLL) return TS_ERR_UNSUPPORTED_SIZE;
   cudaStream_t s = (cudaStream_t)stream;
-  const GlaExtra x = {kscale, decay_scalar, groups, ev, slot_stride, reinterpret_cast<const float2*>(rotation), half};
+  const GlaExtra x = {kscale, decay_scalar ? 1 : 0, groups, ev, slot_stride};
   if (act_dtype == TS_DTYPE_F32)
     return dispatch_gla_scan<float>(q, k, v, ld_qkv, decay, q_scale, state, state_slots, cu_seqlens, o, B, H, d, e, segs, seg_len, scratch, s, x);
   if (act_dtype == TS_DTYPE_BF16)

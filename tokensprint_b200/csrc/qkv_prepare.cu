@@ -24,9 +24,6 @@
 // gate_rows:    y[t, h*e + i] = a[t, h, i] * sigmoid(g[t, h*e + i]) (a has rows of D >= e entries per
 //               head; g null: a plain compaction), the gate in float32; per_head: one gate for a whole
 //               head, g[t, h].
-// rotate_qkv:   out[t] = [rotated q | rotated k | v] in float32 from columns of one product's result: the
-//               first `rot` entries of every head of q and k turn by the table (pairs (i, i + rot/2)), the rest
-//               and the values pass; for recurrences over rotated keys, which take float32 rows.
 #include "common.cuh"
 
 #define QP_WARPS 4
@@ -167,13 +164,19 @@ __global__ void gate_rows_kernel(const TA* __restrict__ a, const TA* __restrict_
 // that fill their rows (D = e), row widths and strides that are multiples of 8.  The sigmoid uses the
 // fast exponential and division: their error disappears in the rounding to bfloat16.
 __global__ void __launch_bounds__(128) gate_rows_vec_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __restrict__ g,
-                                                            long long ld_g, __nv_bfloat16* __restrict__ y, int T, int He) {
+                                                            long long ld_g, __nv_bfloat16* __restrict__ y, int T, int He, int head_e) {
   ts_pdl_prologue();
   const int c = (blockIdx.x * 128 + threadIdx.x) * 8;
   if (c >= He) return;
   for (int t = blockIdx.y; t < T; t += gridDim.y) {
     const uint4 av = *reinterpret_cast<const uint4*>(a + (size_t)t * He + c);
-    const uint4 gv = *reinterpret_cast<const uint4*>(g + (size_t)t * ld_g + c);
+    uint4 gv;
+    if (head_e > 0) {  // one gate for a whole head of head_e entries
+      const __nv_bfloat162 one = __bfloat162bfloat162(g[(size_t)t * ld_g + c / head_e]);
+      gv.x = gv.y = gv.z = gv.w = *reinterpret_cast<const unsigned*>(&one);
+    } else {
+      gv = *reinterpret_cast<const uint4*>(g + (size_t)t * ld_g + c);
+    }
     const __nv_bfloat162 *ah = reinterpret_cast<const __nv_bfloat162*>(&av), *gh = reinterpret_cast<const __nv_bfloat162*>(&gv);
     uint4 ov;
     __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&ov);
@@ -193,52 +196,14 @@ TS_EXPORT int ts_gate_rows(const void* a, const void* g, long long ld_g, int act
   const unsigned blocks = (unsigned)min((n + 255) / 256, (long long)148 * 16);
   cudaStream_t s = (cudaStream_t)stream;
   const int He = H * e;
-  if (act_dtype == TS_DTYPE_BF16 && g != nullptr && !per_head && D == e && He % 8 == 0 && ld_g % 8 == 0 && (((uintptr_t)a | (uintptr_t)g | (uintptr_t)y) & 15) == 0)
+  const bool gate_fits = per_head ? e % 8 == 0 : ld_g % 8 == 0 && ((uintptr_t)g & 15) == 0;
+  if (act_dtype == TS_DTYPE_BF16 && g != nullptr && D == e && He % 8 == 0 && gate_fits && (((uintptr_t)a | (uintptr_t)y) & 15) == 0)
     return ts_launch(gate_rows_vec_kernel, dim3((unsigned)((He / 8 + 127) / 128), (unsigned)min(T, 65535)), dim3(128), 0, s, (const __nv_bfloat16*)a,
-                     (const __nv_bfloat16*)g, ld_g, (__nv_bfloat16*)y, T, He);
+                     (const __nv_bfloat16*)g, ld_g, (__nv_bfloat16*)y, T, He, per_head ? e : 0);
   if (act_dtype == TS_DTYPE_F32)
     return ts_launch(gate_rows_kernel<float>, dim3(blocks), dim3(256), 0, s, (const float*)a, (const float*)g, ld_g, (float*)y, n, H, e, D, per_head);
   if (act_dtype == TS_DTYPE_BF16)
     return ts_launch(gate_rows_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, s, (const __nv_bfloat16*)a, (const __nv_bfloat16*)g, ld_g,
                      (__nv_bfloat16*)y, n, H, e, D, per_head);
-  return TS_ERR_BAD_ARGUMENT;
-}
-
-// One block per token; a thread takes entries of the row [q | k | v] one block width apart.
-template <typename TA>
-__global__ void __launch_bounds__(256) rotate_qkv_kernel(const TA* __restrict__ proj, long long ld, int q_off, int k_off, int v_off,
-                                                         const float2* __restrict__ table, int half, float* __restrict__ out, int Hd, int d, int He) {
-  ts_pdl_prologue();
-  const int t = blockIdx.x;
-  const TA* row = proj + (size_t)t * ld;
-  float* o = out + (size_t)t * (2 * Hd + He);
-  const float2* cs_row = table + (size_t)t * half;
-  for (int i = threadIdx.x; i < Hd; i += blockDim.x) {
-    const int c = i % d;
-    float q = ts_to_float(row[q_off + i]), k = ts_to_float(row[k_off + i]);
-    if (c < 2 * half) {
-      const bool low = c < half;
-      const int other = low ? i + half : i - half;
-      const float2 cs = cs_row[low ? c : c - half];
-      const float sn = low ? -cs.y : cs.y;
-      q = q * cs.x + ts_to_float(row[q_off + other]) * sn;
-      k = k * cs.x + ts_to_float(row[k_off + other]) * sn;
-    }
-    o[i] = q, o[Hd + i] = k;
-  }
-  for (int i = threadIdx.x; i < He; i += blockDim.x) o[2 * Hd + i] = ts_to_float(row[v_off + i]);
-}
-
-TS_EXPORT int ts_rotate_qkv(const void* proj, int act_dtype, long long ld, int q_off, int k_off, int v_off, const float* table, int rot, float* out,
-                            int T, int H, int d, int e, void* stream) {
-  if (T <= 0) return 0;
-  if (H <= 0 || d <= 0 || e <= 0 || rot < 0 || rot > d || (rot & 1) || (rot > 0 && table == nullptr)) return TS_ERR_BAD_ARGUMENT;
-  cudaStream_t s = (cudaStream_t)stream;
-  const float2* tb = reinterpret_cast<const float2*>(table);
-  if (act_dtype == TS_DTYPE_F32)
-    return ts_launch(rotate_qkv_kernel<float>, dim3(T), dim3(256), 0, s, (const float*)proj, ld, q_off, k_off, v_off, tb, rot / 2, out, H * d, d, H * e);
-  if (act_dtype == TS_DTYPE_BF16)
-    return ts_launch(rotate_qkv_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, s, (const __nv_bfloat16*)proj, ld, q_off, k_off, v_off, tb, rot / 2, out,
-                     H * d, d, H * e);
   return TS_ERR_BAD_ARGUMENT;
 }

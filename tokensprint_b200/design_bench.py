@@ -264,10 +264,10 @@ def _vepevik_rooflines(design: str, s: dict, m: dict, peaks: dict) -> dict[str, 
     chans = H * (2 * dd + dv)
     attention_names = ("attention_prefill_tcgen05", "attention_paged_mma", "attention_paged_simple")
     if design == "vepevik":
-        scans = {"linear_scan": (1, H * gd * gv, 6.0), "delta_scan": (1, H * dd * dv, 8.0)}  # layers, state entries, operations
+        scans = {"retention_scan": (1, H * gd * gv, 6.0), "delta_scan": (1, H * dd * dv, 8.0)}  # layers, state entries, operations
         small = {  # bytes per token
             "add_rmsnorm": (2 * s["layers"]) * W * 12 + W * 8, "qkv_prepare": 2 * 2 * (H + 16) * 128 * 2 + 8 * 128 * 2, "gate_rows": 2 * 2 * H * 128 * 2,
-            "rotate_qkv": H * (2 * gd + gv) * (2 + 4), "causal_conv": chans * (2 + 4), "channel_decay": H * dd * 8,
+            "causal_conv": chans * (2 + 4), "channel_decay": H * dd * 8,
             "gla_norm_gate": H * gv * (4 + 2 + 2) + H * dv * (4 + 4 + 2), "capped_glu": 3 * s["top"] * s["expert_ff"] * 2,
             "moe_combine": 3 * (s["top"] + 1) * W * 2, "router": 3 * W * 2,
         }

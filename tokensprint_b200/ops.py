@@ -811,7 +811,7 @@ def gla_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.Te
 
 _SIGNATURES.update({
     "ts_linear_scan": [_c_void_p, _c_void_p, _c_void_p, _c_ll, _c_int, _c_void_p, _c_int, _c_void_p, _c_float, _c_void_p, _c_ll, _c_void_p,
-                       _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p],
+                       _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
     "ts_rows_dot_f32": [_c_void_p, _c_int, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
     "ts_mlstm_gate_scan": [_c_void_p, _c_void_p, _c_float, _c_void_p, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p],
     "ts_mlstm_norm_gate": [_c_void_p, _c_void_p, _c_void_p, _c_ll, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_void_p],
@@ -825,13 +825,14 @@ _SIGNATURES.update({
     "ts_qkv_prepare": [_c_void_p, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_float,
                        _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_float, _c_int,
                        _c_void_p, _c_void_p, _c_void_p, _c_ll, _c_float, _c_void_p],
-    "ts_rotate_qkv": [_c_void_p, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "ts_softcap_rows": [_c_void_p, _c_ll, _c_float, _c_void_p],
     "ts_causal_conv": [_c_void_p, _c_int, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                        _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "ts_delta_scan": [_c_void_p, _c_ll, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_ll, _c_void_p, _c_ll, _c_int, _c_int, _c_void_p, _c_void_p,
                       _c_void_p, _c_ll, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int,
                       _c_void_p],
+    "ts_retention_scan": [_c_void_p, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_ll, _c_void_p, _c_void_p,
+                          _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p],
     "ts_channel_decay": [_c_void_p, _c_ll, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
     "ts_gate_rows": [_c_void_p, _c_void_p, _c_ll, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "ts_weighted_sum": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_float, _c_float, _c_float, _c_float, _c_int, _c_void_p, _c_int, _c_ll,
@@ -847,19 +848,16 @@ def _matrix_view(name: str, t: torch.Tensor, rows: int, cols: int, dtype: Option
 
 def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, kscale: Optional[torch.Tensor], q_scale: float,
                 state: torch.Tensor, state_slots: torch.Tensor, cu_seqlens: torch.Tensor, out: torch.Tensor, num_seqs: int, num_heads: int,
-                groups: int, key_dim: int, value_dim: int, normaliser: bool = False, max_seqlen: Optional[int] = None,
-                rotation: Optional[torch.Tensor] = None) -> None:
+                groups: int, key_dim: int, value_dim: int, normaliser: bool = False, max_seqlen: Optional[int] = None) -> None:
     """S_t = a_t S_(t-1) + (b_t k_t) v_t^T,  out_t = S_t^T (q_t * q_scale), per head, over the step's tokens
-    sequence by sequence, with one decay a_t per (token, head), or (decay [H]) one constant per head.
+    sequence by sequence, with one decay a_t per (token, head).
 
     q, k [T, groups*d] (head h reads group h // (H // groups)) and v [T, H*e]: views with one common
     row stride, float32 or bfloat16 (all three alike); decay [T, H] and kscale [T, H] (or None) float32.
     state [slots, n] float32 with n >= H*d*e': a request's [H, d, e'] block stands at the start of its
     row, e' = e + 1 with `normaliser` (the extra column is fed the value 1 in every token, so it holds
     the sum of the decayed b_t k_t, and its read-out arrives as column e of out), else e' = e.
-    out [T, H*e'] float32.  Long portions run in segments side by side as in gla_scan.
-    `rotation` [T, r/2, 2] float32 (rope_table), in steps of one token per sequence only (max_seqlen = 1): the first r
-    entries of every q and k head turn by it as they are read; longer portions bring rotated rows (rotate_qkv)."""
+    out [T, H*e'] float32.  Long portions run in segments side by side as in gla_scan."""
     flush_gemm_chain()
     H, G, d, e = int(num_heads), int(groups), int(key_dim), int(value_dim)
     ee = e + 1 if normaliser else e
@@ -876,16 +874,9 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.
     _cuda_contig("decay", decay, torch.float32)
     if kscale is not None:
         _cuda_contig("kscale", kscale, torch.float32)
-    constant = decay.dim() == 1
-    for name, t, shape in (("decay", decay, (H,) if constant else (T, H)), ("kscale", kscale, (T, H))):
-        if t is not None and tuple(t.shape) != shape:
-            raise KernelError(f"linear_scan: {name} must be {list(shape)}, got {tuple(t.shape)}")
-    half = 0
-    if rotation is not None:
-        _cuda_contig("rotation", rotation, torch.float32)
-        half = rotation.shape[1]
-        if max_seqlen != 1 or rotation.dim() != 3 or rotation.shape[0] < T or rotation.shape[2] != 2 or 2 * half > d:
-            raise KernelError(f"linear_scan: a rotation is [T, r/2, 2] with r <= {d} and comes in steps of one token, got {tuple(rotation.shape)}")
+    for name, t in (("decay", decay), ("kscale", kscale)):
+        if t is not None and tuple(t.shape) != (T, H):
+            raise KernelError(f"linear_scan: {name} must be [{T}, {H}], got {tuple(t.shape)}")
     _cuda_contig("state_slots", state_slots, torch.int32)
     _cuda_contig("cu_seqlens", cu_seqlens, torch.int32)
     _cuda_contig("out", out, torch.float32)
@@ -903,9 +894,9 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.
         need = int(num_seqs) * segs * H * d * ee + int(num_seqs) * segs * H * d + int(num_seqs) * H * d * ee
         scratch = torch.empty(need, device=q.device, dtype=torch.float32)
     _check("linear_scan", _fn("ts_linear_scan")(
-        q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), _act_code("q", q), decay.data_ptr(), 2 if constant else 1, _ptr(kscale),
+        q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), _act_code("q", q), decay.data_ptr(), 1, _ptr(kscale),
         float(q_scale), state.data_ptr(), state.stride(0), state_slots.data_ptr(), cu_seqlens.data_ptr(), out.data_ptr(), int(num_seqs), H, G, d, e,
-        ee, segs, seg_len, _ptr(scratch), _ptr(rotation), half, _stream()))
+        ee, segs, seg_len, _ptr(scratch), _stream()))
     if segs > 1:
         global launch_count
         launch_count += 1  # the recurrence ran as two kernels
@@ -1229,6 +1220,46 @@ def delta_scan(x: torch.Tensor, q_off: int, k_off: int, v_off: int, beta: torch.
         _stream()))
 
 
+def retention_scan(x: torch.Tensor, q_off: int, k_off: int, v_off: int, rotation: Optional[torch.Tensor], decay: torch.Tensor, q_scale: float,
+                   state: torch.Tensor, state_slots: torch.Tensor, cu_seqlens: torch.Tensor, out: torch.Tensor, num_seqs: int, num_heads: int,
+                   num_qk_heads: int, key_dim: int, value_dim: int, max_seqlen: Optional[int] = None) -> None:
+    """S <- decay_h S + k v^T, out = q_scale S^T q per head over the tokens of every sequence, in order, with one constant
+    decay per head (csrc/delta_rule.cu).  x [T, n] float32 or bfloat16 holds q (columns q_off.., num_qk_heads *
+    key_dim), k (k_off..) and v (v_off.., num_heads * value_dim); with `rotation` [T, r/2, 2] float32 (rope_table) the first
+    r entries of every q and k head turn by it as they are read, pairs r/2 apart.  decay [heads] float32;
+    state, slots and `max_seqlen` as in delta_scan; out [T, heads * value_dim] float32.  Everything but the loads is
+    float32."""
+    flush_gemm_chain()
+    H, G, d, e = int(num_heads), int(num_qk_heads), int(key_dim), int(value_dim)
+    T = x.shape[0]
+    if not x.is_cuda or x.dim() != 2 or x.stride(1) != 1:
+        raise KernelError("retention_scan: x must be a CUDA matrix with unit inner stride")
+    if d > DELTA_MAX_KEY_DIM or G < 1 or H % G:
+        raise KernelError(f"retention_scan: key_dim at most {DELTA_MAX_KEY_DIM}, heads a multiple of the q/k heads")
+    if max(q_off, k_off) + G * d > x.shape[1] or v_off + H * e > x.shape[1]:
+        raise KernelError("retention_scan: the column ranges do not fit x")
+    _cuda_contig("decay", decay, torch.float32)
+    _cuda_contig("out", out, torch.float32)
+    _cuda_contig("state_slots", state_slots, torch.int32)
+    _cuda_contig("cu_seqlens", cu_seqlens, torch.int32)
+    if decay.numel() != H or out.shape != (T, H * e):
+        raise KernelError("retention_scan: one decay per head, out must be [T, heads * value_dim]")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < H * d * e:
+        raise KernelError(f"retention_scan: the state must be float32 [slots, >= {H * d * e}], got {tuple(state.shape)}")
+    if state_slots.numel() < num_seqs or cu_seqlens.numel() < num_seqs + 1:
+        raise KernelError("retention_scan: state_slots and cu_seqlens are shorter than the batch")
+    half = 0
+    if rotation is not None:
+        _cuda_contig("rotation", rotation, torch.float32)
+        if rotation.dim() != 3 or rotation.shape[0] < T or rotation.shape[2] != 2 or 2 * rotation.shape[1] > d:
+            raise KernelError(f"retention_scan: the rotation must be [T, r/2, 2] with r <= {d}, got {tuple(rotation.shape)}")
+        half = rotation.shape[1]
+    _check("retention_scan", _fn("ts_retention_scan")(
+        x.data_ptr(), _act_code("x", x), x.stride(0), int(q_off), int(k_off), int(v_off), _ptr(rotation), half, decay.data_ptr(), state.data_ptr(),
+        state.stride(0), state_slots.data_ptr(), cu_seqlens.data_ptr(), out.data_ptr(), int(num_seqs), H, G, d, e, float(q_scale),
+        1 if max_seqlen == 1 else 0, _stream()))
+
+
 WEIGHTED_SUM_MAX_INPUTS = 4
 
 
@@ -1334,29 +1365,6 @@ def qkv_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_bias: 
         _ptr(table), rot, 1 if unit_norm else 0, float(eps), q_out.data_ptr(), _ptr(k_dst), _ptr(v_dst), _ptr(slot_mapping), T, nq, kv_heads,
         d, e, D, _ptr(positions) if qt_every else None, qt_coef, qt_every, _ptr(q_norm), _ptr(k_norm), _ptr(first_values),
         0 if first_values is None else first_values.stride(0), float(value_share), _stream()))
-
-
-def rotate_qkv(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, table: Optional[torch.Tensor], num_heads: int, key_dim: int,
-               value_dim: int) -> torch.Tensor:
-    """[T, 2*H*d + H*e] float32: the q, k (rotated by the table over the first 2*table.shape[1] entries of every
-    head, pairs half a rotated width apart; None: as they are) and v columns of one projection's result."""
-    flush_gemm_chain()
-    H, d, e = int(num_heads), int(key_dim), int(value_dim)
-    if not proj.is_cuda or proj.dim() != 2 or proj.stride(1) != 1:
-        raise KernelError("rotate_qkv: proj must be a CUDA matrix with unit inner stride")
-    T = proj.shape[0]
-    if max(q_off, k_off) + H * d > proj.shape[1] or v_off + H * e > proj.shape[1]:
-        raise KernelError("rotate_qkv: the column ranges do not fit proj")
-    rot = 0
-    if table is not None:
-        _cuda_contig("table", table, torch.float32)
-        rot = 2 * table.shape[1]
-        if table.dim() != 3 or table.shape[0] < T or table.shape[2] != 2 or rot > d:
-            raise KernelError(f"rotate_qkv: the table must be [T, rot/2, 2] with rot <= {d}, got {tuple(table.shape)}")
-    out = torch.empty((T, 2 * H * d + H * e), device=proj.device, dtype=torch.float32)
-    _check("rotate_qkv", _fn("ts_rotate_qkv")(proj.data_ptr(), _act_code("proj", proj), proj.stride(0), int(q_off), int(k_off), int(v_off),
-                                              _ptr(table), rot, out.data_ptr(), T, H, d, e, _stream()))
-    return out
 
 
 def gate_rows(a: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, num_heads: int, value_dim: int, padded_dim: int,
@@ -2667,7 +2675,7 @@ _TIMED = ("embed_gather", "feed_tokens", "add_rmsnorm", "residual_add", "swiglu"
           "router_topk", "router", "moe_plan", "moe_gate_up", "moe_down", "moe_combine", "branch_norm_add", "stream_add",
           "qk_joint_norm_rope_store", "gla_scan", "gla_norm_gate", "linear_scan", "rows_dot_f32", "mlstm_gate_scan", "mlstm_norm_gate",
           "ssm_conv", "ssm_gate_norm", "scale_rows", "weighted_sum", "rope_table", "qkv_prepare", "gate_rows", "causal_conv", "delta_scan",
-          "channel_decay", "rotate_qkv",
+          "channel_decay", "retention_scan",
           "softcap_rows", "rglru_scan", "rglru_step", "rmsnorm_rows", "library_bmm_float32")
 _plain_functions: dict[str, object] = {}
 _kernel_events: list[tuple[str, "torch.cuda.Event", "torch.cuda.Event"]] = []

@@ -125,10 +125,9 @@ class Retention(Mixer):
 
     Parameters: `hidden_size`, `num_heads`, `key_dim`, `value_dim`, `decay` (a constant per head), `norm_eps`,
     `position` (a position-encoding spec whose rotation pairs entries half a width apart, or None), `k_scale`
-    (default key_dim^-0.5; it goes onto the read-out, in which k is a factor) and the tensors' names.  One product gives [q | k | v | gate].  Rotation, state,
-    recurrence and head norm are float32 whatever the compute dtype: a step of one token per sequence
-    rotates q and k as the recurrence reads them, longer portions bring float32 rows (ops.rotate_qkv).
-    The state is carried from step to step in the request's slot, so prompts may be cut anywhere."""
+    (default key_dim^-0.5; it goes onto the read-out, in which k is a factor) and the tensors' names.  One product
+    gives [q | k | v | gate]; the recurrence's kernel rotates q and k as it reads them.  Rotation, state, recurrence
+    and head norm are float32 whatever the compute dtype.  The state ([heads, e, d]) is carried from step to step in the request's slot, so prompts may be cut anywhere."""
 
     graph_safe = True
     reads_through_ops = True
@@ -140,8 +139,8 @@ class Retention(Mixer):
         self.norm_eps = float(norm_eps)
         if min(self.num_heads, self.key_dim, self.value_dim) < 1 or len(decay) != self.num_heads:
             raise ValueError("retention: sizes must be positive and there is one decay per head")
-        if self.key_dim > ops.GLA_MAX_KEY_DIM:
-            raise ValueError(f"retention: key_dim {key_dim} exceeds the kernel's {ops.GLA_MAX_KEY_DIM}")
+        if self.key_dim > ops.DELTA_MAX_KEY_DIM:
+            raise ValueError(f"retention: key_dim {key_dim} exceeds the kernel's {ops.DELTA_MAX_KEY_DIM}")
         self.k_scale = float(k_scale) if k_scale is not None else float(self.key_dim) ** -0.5
         self.position = build_part("position_encoding", position, ctx) if position is not None else None
         if self.position is not None and (not hasattr(self.position, "rotary_table") or self.position.pairing != "half"
@@ -181,14 +180,9 @@ class Retention(Mixer):
         hd, he = H * d, H * e
         proj = linear(x, self.in_weight, next_weight=self.o_weight)
         table = self.position.rotary_table(step) if self.position is not None else None
-        if step.max_seqlen_q == 1:
-            rows, rotation = proj, table
-        else:
-            rows, rotation = ops.rotate_qkv(proj, 0, hd, 2 * hd, table, H, d, e), None
-        q, k, v = rows[:, :hd], rows[:, hd:2 * hd], rows[:, 2 * hd:2 * hd + he]
         o = torch.empty((T, he), device=x.device, dtype=torch.float32)
-        ops.linear_scan(q, k, v, self.decay, None, self.k_scale, cache.state, step.state_slots, step.cu_seqlens_q, o, step.num_seqs, H, H, d, e,
-                        max_seqlen=step.max_seqlen_q, rotation=rotation)
+        ops.retention_scan(proj, 0, hd, 2 * hd, table, self.decay, self.k_scale, cache.state, step.state_slots, step.cu_seqlens_q, o, step.num_seqs,
+                           H, H, d, e, max_seqlen=step.max_seqlen_q)
         y = torch.empty((T, he), device=x.device, dtype=x.dtype)
         ops.gla_norm_gate(o, proj[:, 2 * hd + he:], None, y, H, e, self.norm_eps)
         return linear(y, self.o_weight, next_weight=step.weight_after)
