@@ -6,8 +6,8 @@
 //                 sigmoid(logit), handed on as they are or divided by their sum (`renormalize`), or
 //                 the softmax over the chosen logits alone (`score_mode`); or, with the softmax over all
 //                 logits as scores, the `top` largest of score + correction (a number per expert that
-//                 steers the choice only) with the scores themselves as weights.  Experts may form equal groups of
-//                 neighbours: only those of the groups with the best members are then chosen.  A constant
+//                 steers the choice only) with the scores themselves as weights.  The list of experts
+//                 may be cut into runs of one length: the choice is then made among the runs with the best members.  A constant
 //                 may multiply the weights.
 //   moe_plan    : the (token, choice) pairs sorted by expert: offsets[e] .. offsets[e+1] are expert
 //                 e's places in `order` (pair indices), tile_offsets[e] its first row tile of
@@ -37,8 +37,8 @@
 
 // What a router may do beyond scores and a choice of the largest.
 struct RouterGroups {
-  int count;    // experts form `count` equal groups of neighbours (0 or 1: no groups)
-  int keep;     // only experts of the `keep` groups whose best member is largest may be chosen
+  int count;    // the list of experts is cut into `count` runs of one length (0 or 1: it is not)
+  int keep;     // the choice is made among the `keep` runs with the largest best members
   float scale;  // a constant on every weight, after they are divided by their sum
 };
 

@@ -1546,8 +1546,8 @@ def router_topk(logits: torch.Tensor, top: int, renormalize: bool, ids: torch.Te
     weights are sigmoid(logit) (divided by their sum if `renormalize`); "softmax_chosen": the softmax
     over the chosen logits alone; "softmax_all": the scores are the softmax over all E logits, the
     `top` largest of score + correction [E] are chosen, and the weights are the scores themselves (divided by
-    their sum if `renormalize`).  groups (count, keep): experts form `count` equal groups of neighbours, and only those
-    of the `keep` groups whose best member is largest may be chosen.  scale: a constant on all weights."""
+    their sum if `renormalize`).  groups (count, keep): the list of experts is cut into `count` runs of one length, and
+    the choice is made among the `keep` runs with the largest best members.  scale: a constant on all weights."""
     flush_gemm_chain()
     _cuda_contig("logits", logits, torch.float32)
     _cuda_contig("ids", ids, torch.int32)

@@ -91,8 +91,8 @@ class RoutedExperts(FeedForward):
                  "softmax_all": scores s = softmax(z) over all experts; the `top` largest of
                  s + c are chosen (`correction` names c, a number per expert that steers the choice
                  only) and the weights are the chosen s themselves (divided by their sum with `renormalize`)
-        `groups` = (count, keep): the experts form `count` equal groups of neighbours; only those of the `keep` groups
-                    whose best member is largest may be chosen
+        `groups` = (count, keep): the list of experts is cut into `count` runs of one length and the choice is made among
+                    the `keep` runs with the largest best members
         `weight_scale`: a constant on every weight, after the division by their sum
         f = sum over chosen e of expert_e(w_e x)   (`weight_on` "input"; "output": w_e expert_e(x))
             + shared(x) if a shared expert is named (any feed-forward spec)
